@@ -382,15 +382,19 @@ int b200_lm_rope_table(const int* pos, const double* inv_freq, float* cs, int T,
 /* n = y / sqrt(mean(y^2) + eps) * (w_offset + w); x = n or (add) x += n.  wgt != NULL: y row t is the weighted
  * sum of rows t*top .. t*top+top-1 of y.  rows != NULL: the input row of output t is rows[t].  center: y's mean is
  * taken off first (a layer norm without bias).
- * groups > 1: the row is `groups` equal consecutive parts, each with its own root mean square (no centering) */
+ * groups > 1: the row is `groups` equal consecutive parts, each with its own root mean square (no centering);
+ * bias (bf16 [N], may be NULL): added after the weight */
 int b200_lm_norm_rows(const float* y, long ldy, const float* wgt, int top, const void* w, float w_offset, float eps,
-                      float* x, long ldx, int add, const int* rows, int center, int groups, int T, int N, void* stream);
+                      float* x, long ldx, int add, const int* rows, int center, int groups, const void* bias, int T, int N,
+                      void* stream);
 /* the residual update of b200_lm_residual_rows on res (stored back) followed by the norm of the updated row into out:
- * res[t] += ls * mult * (...); out[t] = norm(res[t]) * (w_offset + w), the norm in `groups` parts */
+ * res[t] = keep * res[t] + ls * mult * (...); out[t] = norm(res[t]) * (w_offset + w) + bias, the norm in `groups` parts.
+ * out may be res itself (a stream that is normed after every sum: the row is written once, normed).  out_bf16 (may be
+ * NULL): the result also as bf16 rows of ldb >= N columns, zero-padded (the operand of the next product) */
 int b200_lm_residual_norm_rows(const float* y, long ldy, const float* wgt, int top, const float* shared, long lds,
                                const float* sgate, long ldsg, const void* ls, float* res, long ldr, const void* w,
                                float w_offset, float eps, int center, float* out, long ldo, int groups, float mult,
-                               int T, int N, void* stream);
+                               const void* bias, float keep, void* out_bf16, long ldb, int T, int N, void* stream);
 /* D[t] = [q latent | kv latent | rotated key part] (the fused down-projection): cq = rmsnorm(q latent) * wq;
  * own_kv: rmsnorm(kv latent) * wkv and the rotated part go to cache[slot[t]][pos[t]] = [kv_rank | rot_dim] */
 int b200_lm_latent_post(const float* D, long ldd, const void* wq, const void* wkv, float eps, float* cq, long ldq,
@@ -482,6 +486,12 @@ int b200_lm_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* 
                      int dim, int vdim, int rot_dims, const void* qn_w, const void* kn_w, float eps, int v_unit, float qt_coef,
                      int qt_every, const void* vmix, const float* v_first, long ldvf, float* v_keep, long ldvk, int T,
                      void* stream);
+/* the same step with everything per head: qn_w / kn_w (bf16 [dim], or NULL): RMS norm (eps) of every query / key head times
+ * ONE weight for all heads; then the rotation of pairs (i, i + rot_dims / 2) or (pairs) (2i, 2i + 1); V may be K's own rows */
+int b200_lm_head_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* V, long ldv, void* cache, int cache_bf16,
+                          long slot_stride, long tok_stride, const int* slot, const int* pos, const float* cs, int H, int G,
+                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int T,
+                          void* stream);
 /* out[t][h] = softmax over the visible rows j of slot[t] (and the sink logit of head h, if any) of
  * scale * q[t][h] . K_j[h / (H/G)], times V_j; visible: max(block start of pos[t] (chunk > 0), pos[t] - window + 1
  * (window > 0), 0) <= j <= pos[t].  bias_exp > 0: 2^(-bias_exp (h + 1) / H) (pos[t] - j) is taken off the score;
@@ -501,13 +511,17 @@ int b200_lm_sink_attention(const float* q, long ldq, const void* cache, int cach
  * With it, prep and n_parts > 1: every sequence is walked in parts of part_len tokens at the same time (the state is linear
  * in its start: a first pass leaves every part's own contribution and decay product, a small launch chains them into the
  * parts' start states, a second pass walks every part from its start state); n_parts >= the parts of the longest
- * sequence, part_scratch: n_seq * n_parts * (H * 8 * vdim * lanes + H * lanes * 8) floats, lanes = the state layout's */
+ * sequence, part_scratch: n_seq * n_parts * (H * 8 * vdim * lanes + H * lanes * 8) floats, lanes = the state layout's.
+ * wraw with delta: the delta rule with a decay per key channel, S <- diag(w) S; S <- S + k (beta (v - S^T k))^T; out = S^T q,
+ * w = exp(-exp(A_log[h]) softplus(wraw + dt_bias[h dim + i])); with prep the sequences are walked 8 tokens at a time
+ * (max_rows: the rows of the longest sequence; prep: (T / 8 + n_seq + 1) * H * (25 * 8 lanes + 128) floats, 16-byte aligned) */
 int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv, float* out, long ldo,
                          float* state, long slot_stride, const int* seqs, int n_seq, const int* slot, const int* pos,
                          int H, int rep, int dim, int vdim, int act, float unit_eps, float q_scale,
                          const float* decay_const, const float* a, long lda, const void* A_log, const void* dt_bias,
                          const float* b, long ldb, int delta, int dt_in, const void* skip, const float* wraw, long ldwr,
-                         const void* bonus, float* prep, int part_len, int n_parts, float* part_scratch, int T, void* stream);
+                         const void* bonus, float* prep, int part_len, int n_parts, float* part_scratch, int max_rows, int T,
+                         void* stream);
 /* operands of the tensor-core attention of a prompt step: out[(t, r)] = bf16 of q[t][r * dim .. + dim) padded to Kp;
  * P[(t, r)][j] = softmax over the visible keys key0 + j (and sink[r]) of scale * S[(t, r)][j], bf16, zero elsewhere;
  * split: P rows are [hi | lo] (Sp columns each), lo the rounding error of hi (the operand of a two-part product) */
@@ -520,14 +534,15 @@ int b200_lm_sink_softmax_bf16(const float* S, long lds, const int* pos, int rep,
 int b200_lm_head_post(const float* o, long ldi, const float* gate, long ldg, const void* w, int w_len, float eps, int span,
                       int gate_per_head, int gate_silu, int dv, int n, float scale, float* out, long ldo, int gate_first,
                       int T, void* stream);
-/* Y = g sigmoid(alpha (g + cubic g^3)) (u + up_off), g = min(G, limit), u = clamp(U, -limit, limit) */
+/* Y = g sigmoid(alpha (g + cubic g^3)) (u + up_off), g = min(G, limit), u = clamp(U, -limit, limit); relu: the gate passes
+ * max(g, 0) instead */
 int b200_lm_glu_clamp(const float* G, long ldg, const float* U, long ldu, float limit, float alpha, float cubic, float up_off,
-                      float* Y, long ldy, int n, int T, void* stream);
+                      int relu, float* Y, long ldy, int n, int T, void* stream);
 
 /* the same as bf16 rows of Kp >= n columns (zero-padded): the operand of the next tensor-core product; live != NULL:
  * rows t with live[t] < 0 (the padding of sorted expert segments) are written as zeros and their inputs are not read */
 int b200_lm_glu_clamp_bf16(const float* G, long ldg, const float* U, long ldu, float limit, float alpha, float cubic, float up_off,
-                           void* Y, int n, int Kp, const int* live, int T, void* stream);
+                           int relu, void* Y, int n, int Kp, const int* live, int T, void* stream);
 
 #ifdef __cplusplus
 }

@@ -82,6 +82,10 @@ struct NormP {
   const float* sgate; long ldsg;
   int groups;                         // parts of the row with a root mean square of their own (1: the whole row)
   float mult;                         // the residual update is scaled by this number as well (beside ls)
+  const bf16* bias;                   // [N] or NULL: added after the weight (one group only)
+  float keep;                         // the residual row itself counts this often: res = keep * res + ls * mult * (...).  When
+                                      // x is res (a norm of the sum), the row is written once, normed
+  bf16* xb; long ldb;                 // != NULL: the result also as bf16 operand rows of ldb >= N columns (zero padding)
 };
 __global__ void norm_rows_kernel(NormP p) {
   extern __shared__ float sm[];
@@ -102,8 +106,8 @@ __global__ void norm_rows_kernel(NormP p) {
     if (p.res) {                      // the same arithmetic, in the same order, as residual_rows_kernel
       if (p.shared) v = fmaf(sg, p.shared[r * p.lds + i], v);
       float* o = p.res + r * p.ldr + i;
-      v = fmaf((p.ls ? bf2f(p.ls[i]) : 1.f) * p.mult, v, *o);
-      *o = v;
+      v = fmaf((p.ls ? bf2f(p.ls[i]) : 1.f) * p.mult, v, p.keep * *o);
+      if (p.res != p.x) *o = v;
     }
     row[i] = v;
     ss += p.center ? v : v * v;
@@ -135,10 +139,14 @@ __global__ void norm_rows_kernel(NormP p) {
   }
   const float inv = 1.0f / sqrtf(tot / (float)p.N + p.eps);
   for (int i = threadIdx.x; i < p.N; i += blockDim.x) {
-    const float v = (row[i] - mean) * inv * (p.w_offset + bf2f(p.w[i]));
+    float v = (row[i] - mean) * inv * (p.w_offset + bf2f(p.w[i]));
+    if (p.bias) v += bf2f(p.bias[i]);
     float* o = p.x + (long)t * p.ldx + i;
     *o = p.add ? *o + v : v;
+    if (p.xb) p.xb[(long)t * p.ldb + i] = f2bf(v);
   }
+  if (p.xb)
+    for (int i = p.N + threadIdx.x; i < p.ldb; i += blockDim.x) p.xb[(long)t * p.ldb + i] = f2bf(0.f);
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -1056,13 +1064,15 @@ int b200_lm_rope_table(const int* pos, const double* inv_freq, float* cs, int T,
 }
 
 int b200_lm_norm_rows(const float* y, long ldy, const float* wgt, int top, const void* w, float w_offset, float eps,
-                      float* x, long ldx, int add, const int* rows, int center, int groups, int T, int N, void* st) {
+                      float* x, long ldx, int add, const int* rows, int center, int groups, const void* bias, int T, int N,
+                      void* st) {
   B200_REQUIRE(y && w && x && T > 0 && N > 0, "lm_norm_rows: bad argument");
   if (groups < 1) groups = 1;
+  B200_REQUIRE(!bias || groups == 1, "lm_norm_rows: a bias goes with one group");
   B200_REQUIRE(N % groups == 0 && groups <= 1024 && !(center && groups > 1), "lm_norm_rows: %d parts of a row of %d numbers", groups, N);
   B200_REQUIRE((N + 32 + groups) * 4 <= 48 * 1024, "lm_norm_rows: rows of %d numbers do not fit shared memory", N);
   NormP p{y, ldy, wgt, wgt ? top : 0, (const bf16*)w, w_offset, eps, x, ldx, add, rows, N, center, nullptr, 0, nullptr, nullptr, 0, nullptr, 0,
-          groups, 1.f};
+          groups, 1.f, (const bf16*)bias, 1.f, nullptr, 0};
   norm_rows_kernel<<<T, T < 64 ? 1024 : 256, (N + 32 + groups) * sizeof(float), (cudaStream_t)st>>>(p);
   B200_CHECK_LAUNCH();
   return B200_OK;
@@ -1071,13 +1081,16 @@ int b200_lm_norm_rows(const float* y, long ldy, const float* wgt, int top, const
 int b200_lm_residual_norm_rows(const float* y, long ldy, const float* wgt, int top, const float* shared, long lds,
                                const float* sgate, long ldsg, const void* ls, float* res, long ldr, const void* w,
                                float w_offset, float eps, int center, float* out, long ldo, int groups, float mult,
-                               int T, int N, void* st) {
+                               const void* bias, float keep, void* out_bf16, long ldb, int T, int N, void* st) {
   B200_REQUIRE(y && res && w && out && T > 0 && N > 0 && (top == 0 || wgt), "lm_residual_norm_rows: bad argument");
   if (groups < 1) groups = 1;
+  B200_REQUIRE((!bias && !out_bf16) || groups == 1, "lm_residual_norm_rows: a bias and operand rows go with one group");
+  B200_REQUIRE(!out_bf16 || ldb >= N, "lm_residual_norm_rows: operand rows of %ld columns for %d numbers", ldb, N);
+  B200_REQUIRE(out != res || ldo == ldr, "lm_residual_norm_rows: a result in place has the residual's row pitch");
   B200_REQUIRE(N % groups == 0 && groups <= 1024 && !(center && groups > 1), "lm_residual_norm_rows: %d parts of a row of %d numbers", groups, N);
   B200_REQUIRE((N + 32 + groups) * 4 <= 48 * 1024, "lm_residual_norm_rows: rows of %d numbers do not fit shared memory", N);
   NormP p{y, ldy, wgt, wgt ? top : 0, (const bf16*)w, w_offset, eps, out, ldo, 0, nullptr, N, center,
-          res, ldr, (const bf16*)ls, shared, lds, sgate, ldsg, groups, mult};
+          res, ldr, (const bf16*)ls, shared, lds, sgate, ldsg, groups, mult, (const bf16*)bias, keep, (bf16*)out_bf16, ldb};
   norm_rows_kernel<<<T, T < 64 ? 1024 : 256, (N + 32 + groups) * sizeof(float), (cudaStream_t)st>>>(p);
   B200_CHECK_LAUNCH();
   return B200_OK;

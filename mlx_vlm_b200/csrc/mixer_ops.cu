@@ -24,7 +24,13 @@ __device__ __forceinline__ void st_row(bf16* p, float v) { *p = f2bf(v); }
 __device__ __forceinline__ float sigmoid_exact(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_exact(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float glu_arg(float g, float cubic) { return cubic != 0.f ? g + cubic * g * g * g : g; }
+struct GluP { float lim, alpha, cubic, up_off; int relu; };      // a gated unit: act(min(a, lim)) (clamp(b, +-lim) + up_off)
+__device__ __forceinline__ float glu_unit(float a, float b, const GluP& p) {
+  const float g = fminf(a, p.lim), u = fminf(fmaxf(b, -p.lim), p.lim);
+  if (p.relu) return fmaxf(g, 0.f) * (u + p.up_off);
+  const float arg = p.cubic != 0.f ? g + p.cubic * g * g * g : g;
+  return g * sigmoid_exact(p.alpha * arg) * (u + p.up_off);
+}
 __device__ __forceinline__ float block_sum_fixed(float v, float* red) {
   v = warp_sum(v);
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
@@ -221,6 +227,59 @@ __global__ void qkv_post_kernel(QkvPostP<CT> p) {
       if (p.v_keep) p.v_keep[(long)t * p.ldvk + e] = a;
       st_row(row + p.G * p.dim + e, a);
     }
+  }
+}
+
+// The same step with everything per head: an optional RMS norm of every query and key head with ONE weight vector for all
+// heads, then the rotation (pairs (i, i + rot_dims / 2), or, `pairs`, (2i, 2i + 1)), queries in place and keys into the
+// cache row, values copied behind them (V may be the rows of K itself: K is only read).  A warp per head, so a step of one
+// token still spreads over several blocks.
+template <typename CT>
+struct HeadQkvP {
+  float* Q; long ldq;
+  const float* K; long ldk;
+  const float* V; long ldv;
+  CT* cache; long slot_stride, tok_stride;
+  const int *slot, *pos;
+  const float2* cs;                // [T][rot_dims / 2]
+  int H, G, dim, vdim, rot_dims, pairs;
+  const bf16 *qn_w, *kn_w;         // [dim] or NULL
+  float eps;
+};
+template <typename CT>
+__global__ void head_qkv_post_kernel(HeadQkvP<CT> p) {
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims / 2;
+  const int u = blockIdx.y * (blockDim.x >> 5) + warp;                 // query heads, then key heads, then value heads
+  if (u >= p.H + 2 * p.G) return;
+  CT* row = p.cache + (long)p.slot[t] * p.slot_stride + (long)p.pos[t] * p.tok_stride;
+  if (u >= p.H + p.G) {
+    const int g = u - p.H - p.G;
+    const float* v = p.V + (long)t * p.ldv + (long)g * p.vdim;
+    CT* d = row + (long)p.G * p.dim + (long)g * p.vdim;
+    for (int i = lane; i < p.vdim; i += 32) st_row(d + i, v[i]);
+    return;
+  }
+  const bool query = u < p.H;
+  const int h = query ? u : u - p.H;
+  float* q = p.Q + (long)t * p.ldq + (long)h * p.dim;
+  const float* x = query ? q : p.K + (long)t * p.ldk + (long)h * p.dim;
+  const bf16* w = query ? p.qn_w : p.kn_w;
+  CT* kd = row + (long)h * p.dim;
+  float inv = 1.f;
+  if (w) {
+    float ss = 0.f;
+    for (int i = lane; i < p.dim; i += 32) ss = fmaf(x[i], x[i], ss);
+    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);           // (also: every lane has read the row before one writes)
+  }
+  auto in = [&](int i) { return w ? x[i] * inv * bf2f(w[i]) : x[i]; };
+  auto put = [&](int i, float v) { if (query) q[i] = v; else st_row(kd + i, v); };
+  for (int e = lane; e < half + p.dim - p.rot_dims; e += 32) {         // a lane reads and writes both numbers of its pair
+    if (e >= half) { const int i = e + half; put(i, in(i)); continue; }
+    const int i = p.pairs ? 2 * e : e, j = p.pairs ? 2 * e + 1 : e + half;
+    const float2 a = p.cs[(long)t * half + e];
+    const float lo = in(i), hi = in(j);
+    put(i, lo * a.x - hi * a.y);
+    put(j, hi * a.x + lo * a.y);
   }
 }
 
@@ -439,7 +498,9 @@ struct StateP {
   const bf16* skip;                 // [H] or NULL: o += skip[h] v
   // decay per key channel (the template's CHAN):  o = S^T q + (sum_i q_i bonus_i k_i) v  with S the state BEFORE the
   // token, then  S <- diag(w) S + k v^T.  Prepared: wdec [T][H dim] holds w and kq_in the bracket; else wdec holds the
-  // logits x of w = exp(-exp(x)) and the bracket is made here from `bonus` ([H][dim])
+  // logits x of w = exp(-exp(x)) and the bracket is made here from `bonus` ([H][dim]).
+  // With the delta rule (CHAN and DELTA; q, k shared by `rep` heads): S <- diag(w) S, u = beta (v - S^T k), S <- S + k u^T,
+  // o = S^T q, and wdec holds x of w = exp(-exp(A_log[h]) softplus(x + dt_bias[h dim + i]))
   const float* wdec; long ldw;
   const bf16* bonus;
   // A long sequence in parts that are walked at the same time (decay per key channel, prepared inputs).  The state is
@@ -577,6 +638,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
       const long t = start + c0 + threadIdx.x;
       if (CHAN) {
         if (p.kq_in) rkq = p.kq_in[t * (p.H / p.rep) + hk];
+        if (DELTA) rb = p.b[t * p.ldb + h];
       } else if (p.kq_in) {
         ra = p.dec_in[t * p.H + h]; rb = p.bet_in[t * p.H + h]; rkq = p.kq_in[t * (p.H / p.rep) + hk];
       } else {
@@ -585,7 +647,8 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
       }
     }
   };
-  const float A = (CHAN || p.decay_const || !raw) ? 0.f : expf(bf2f(p.A_log[h])), dtb = (CHAN || p.decay_const || !raw) ? 0.f : bf2f(p.dt_bias[h]);
+  const float A = ((CHAN && !DELTA) || p.decay_const || !raw) ? 0.f : expf(bf2f(p.A_log[h]));
+  const float dtb = (CHAN || p.decay_const || !raw) ? 0.f : bf2f(p.dt_bias[h]);
   const float dconst = p.decay_const ? p.decay_const[h] : 0.f;
   const float skip = p.skip ? bf2f(p.skip[h]) : 0.f;
   request(0);
@@ -598,7 +661,12 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
       if (e < CT * DKP) {
         ks[tk][(i / LS_R) * LS_RS + (i % LS_R)] = act_qk ? silu_exact(rk[n]) : rk[n];
         qs[tk][(i / LS_R) * LS_RS + (i % LS_R)] = act_qk ? silu_exact(rq[n]) : rq[n];
-        if (CHAN) ws[tk][(i / LS_R) * LS_RS + (i % LS_R)] = raw ? expf(-expf(rw[n])) : rw[n];
+        if (CHAN && DELTA) {
+          const float x = i < p.dim ? rw[n] + bf2f(p.dt_bias[(long)h * p.dim + i]) : 0.f;
+          ws[tk][(i / LS_R) * LS_RS + (i % LS_R)] = expf(-A * softplus_exact(x));
+        } else if (CHAN) {
+          ws[tk][(i / LS_R) * LS_RS + (i % LS_R)] = raw ? expf(-expf(rw[n])) : rw[n];
+        }
       }
     }
 #pragma unroll
@@ -609,6 +677,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
     if ((int)threadIdx.x < nc) {
       if (CHAN) {
         if (!raw) kq[threadIdx.x] = rkq;
+        if (DELTA) bet[threadIdx.x] = sigmoid_exact(rb);
       } else if (raw) {
         const float dt = p.decay_const ? 0.f : softplus_exact(ra + dtb);
         dec[threadIdx.x] = p.decay_const ? dconst : expf(-A * dt);
@@ -634,7 +703,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
         const int at = (i / LS_R) * LS_RS + (i % LS_R);
         const float a = ks[tk][at] * ik, b = qs[tk][at] * iq;
         ks[tk][at] = a; qs[tk][at] = b;
-        dot = CHAN ? fmaf(a * b, bf2f(p.bonus[(long)hk * p.dim + i]), dot) : fmaf(a, b, dot);
+        dot = (CHAN && !DELTA) ? fmaf(a * b, bf2f(p.bonus[(long)hk * p.dim + i]), dot) : fmaf(a, b, dot);
       }
       dot = warp_sum(dot);
       if (lane == 0) kq[tk] = dot;
@@ -651,6 +720,29 @@ __global__ void __launch_bounds__(LS_THREADS) linear_state_kernel(StateP p) {
       const float4 q0 = *reinterpret_cast<const float4*>(qp), q1 = *reinterpret_cast<const float4*>(qp + 4);
       const float k_[LS_R] = {k0.x, k0.y, k0.z, k0.w, k1.x, k1.y, k1.z, k1.w};
       const float q_[LS_R] = {q0.x, q0.y, q0.z, q0.w, q1.x, q1.y, q1.z, q1.w};
+      if (CHAN && DELTA) {         // every row decays by itself first; then both dots of the decayed state in one pass
+        const float4 w0 = *reinterpret_cast<const float4*>(wp), w1 = *reinterpret_cast<const float4*>(wp + 4);
+        const float w_[LS_R] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+        wp += LD;
+        float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < LS_R; i += 2) {
+          S[i] *= w_[i]; S[i + 1] *= w_[i + 1];
+          a0 = fmaf(S[i], k_[i], a0); a1 = fmaf(S[i + 1], k_[i + 1], a1);
+          b0 = fmaf(S[i], q_[i], b0); b1 = fmaf(S[i + 1], q_[i + 1], b1);
+        }
+        float dk = a0 + a1, dq = b0 + b1;
+#pragma unroll
+        for (int o = 1; o < P; o <<= 1) {
+          dk += __shfl_xor_sync(0xffffffffu, dk, o);
+          dq += __shfl_xor_sync(0xffffffffu, dq, o);
+        }
+        const float u = bet[tk] * (vs[tk][cj] - dk);
+        if (r == 0 && valid) *op = fmaf(u, kq[tk], dq);
+#pragma unroll
+        for (int i = 0; i < LS_R; ++i) S[i] = fmaf(k_[i], u, S[i]);
+        continue;
+      }
       if (CHAN) {                  // the output reads the state before the token; every row has its own decay
         const float4 w0 = *reinterpret_cast<const float4*>(wp), w1 = *reinterpret_cast<const float4*>(wp + 4);
         const float w_[LS_R] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
@@ -881,6 +973,271 @@ __global__ void state_parts_chain_kernel(StateP p, int P) {
 }
 
 // ---------------------------------------------------------------------------------------------------------
+// The delta rule with a decay per key channel over a prompt, DC_C tokens of a sequence at a time.  With S the state before a
+// chunk, g_t the decays of its tokens, G_t = prod_{s <= t} g_s and, per channel, all products of decays taken over the
+// tokens between two of the chunk (so nothing is ever divided by a decay and every factor is at most 1),
+//   k~_t = G_t k_t,   q~_t = G_t q_t,   k^_t = (prod_{s > t} g_s) k_t,
+//   A_ts = sum_i k_t k_s prod_{s < r <= t} g_r  (s < t),   B_ts = sum_i q_t k_s prod_{s < r <= t} g_r  (s <= t),
+// the token-by-token rule is exactly
+//   u = T (v - S^T k~),  T = (1 + diag(beta) A)^-1 diag(beta),   o = S^T q~ + (B T) (v - S^T k~),   S <- diag(G_C) S + k^ u^T.
+// k~, q~, k^, G_C, T and B T do not depend on S: delta_chunk_prep_kernel makes them for all chunks at once (a warp per chunk
+// and head), delta_chunk_kernel walks the chunks.  The chain from chunk to chunk then holds ONE reduction over the lanes of
+// a column for DC_C tokens, and the 2 DC_C sums of a column are reduced together (each lane ends with its own sums).
+// All arithmetic is fp32.  A chunk past the end of its sequence is filled with tokens that change nothing (g = 1, k = q = 0).
+constexpr int DC_C = 8;
+struct DeltaChunkP {
+  const float* q; long ldq;         // activated
+  const float* k; long ldk;
+  const float* v; long ldv;
+  float* out; long ldo;
+  float* state; long slot_stride;
+  const int* seqs;
+  const int *slot, *pos;
+  int H, rep, dim, vdim;
+  float unit_eps, q_scale;
+  const float* x; long ldx;         // [T][H dim] logits of the decays: g = exp(-exp(A_log[h]) softplus(x + dt_bias))
+  const bf16 *A_log, *dt_bias;      // [H], [H dim]
+  const float* b; long ldb;         // beta = sigmoid(b[t][h])
+  float* tiles;                     // per (chunk, head): k~ [C][D], q~ [C][D], k^ [C][D], G_C [D], T [C][C], B T [C][C]
+};
+// the first chunk of sequence g of the step: no two sequences share one (a sequence has at most rows / C + 1 of them)
+__device__ __forceinline__ long first_chunk(const int* seqs, int g) { return seqs[2 * g] / DC_C + g; }
+template <int P>
+__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(DeltaChunkP p) {
+  constexpr int C = DC_C, D = P * LS_R, NCH = (D + 31) / 32, TILE = (3 * C + 1) * D + 2 * C * C;
+  __shared__ float sA[4][C * C], sB[4][C * C], sT[4][C * C];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, seq = blockIdx.z;
+  const int h = blockIdx.y * 4 + warp, hk = h / p.rep;
+  const int start = p.seqs[2 * seq] + blockIdx.x * C, nc = min(C, p.seqs[2 * seq + 1] - (int)blockIdx.x * C);
+  if (nc <= 0 || h >= p.H) return;             // whole warps
+  float* tile = p.tiles + ((first_chunk(p.seqs, seq) + blockIdx.x) * p.H + h) * TILE;
+  float ik[C], iq[C];
+#pragma unroll
+  for (int t = 0; t < C; ++t) {
+    float sk = 0.f, sq = 0.f;
+    if (t < nc) {
+      const float* kr = p.k + (long)(start + t) * p.ldk + (long)hk * p.dim;
+      const float* qr = p.q + (long)(start + t) * p.ldq + (long)hk * p.dim;
+      for (int i = lane; i < p.dim; i += 32) { sk = fmaf(kr[i], kr[i], sk); sq = fmaf(qr[i], qr[i], sq); }
+    }
+    ik[t] = 1.0f / sqrtf(warp_sum(sk) + p.unit_eps);
+    iq[t] = p.q_scale / sqrtf(warp_sum(sq) + p.unit_eps);
+  }
+  const float A = expf(bf2f(p.A_log[h]));
+  float acc[C * C];                            // entry (t, s): A_ts below the diagonal; B_ts is kept in bcc
+  float bcc[C * C];
+#pragma unroll
+  for (int e = 0; e < C * C; ++e) acc[e] = bcc[e] = 0.f;
+#pragma unroll 1
+  for (int n = 0; n < NCH; ++n) {
+    const int i = n * 32 + lane;
+    float k[C], q[C], g[C];
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      const bool ok = t < nc && i < p.dim;
+      k[t] = ok ? p.k[(long)(start + t) * p.ldk + (long)hk * p.dim + i] * ik[t] : 0.f;
+      q[t] = ok ? p.q[(long)(start + t) * p.ldq + (long)hk * p.dim + i] * iq[t] : 0.f;
+      g[t] = 1.f;
+      if (ok) g[t] = expf(-A * softplus_exact(p.x[(long)(start + t) * p.ldx + (long)h * p.dim + i] + bf2f(p.dt_bias[(long)h * p.dim + i])));
+    }
+#pragma unroll
+    for (int s = 0; s < C; ++s) {
+      float kd = k[s];
+      bcc[s * C + s] = fmaf(q[s], kd, bcc[s * C + s]);
+#pragma unroll
+      for (int t = s + 1; t < C; ++t) {
+        kd *= g[t];
+        acc[t * C + s] = fmaf(k[t], kd, acc[t * C + s]);
+        bcc[t * C + s] = fmaf(q[t], kd, bcc[t * C + s]);
+      }
+      if (i < D) tile[(2 * C + s) * D + i] = kd;
+    }
+    float G = 1.f;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      G *= g[t];
+      if (i < D) { tile[t * D + i] = G * k[t]; tile[(C + t) * D + i] = G * q[t]; }
+    }
+    if (i < D) tile[3 * C * D + i] = G;
+  }
+#pragma unroll
+  for (int t = 0; t < C; ++t)
+#pragma unroll
+    for (int s = 0; s <= t; ++s) {
+      const float a = s < t ? warp_sum(acc[t * C + s]) : 0.f, b = warp_sum(bcc[t * C + s]);
+      if (lane == 0) { sA[warp][t * C + s] = a; sB[warp][t * C + s] = b; }
+    }
+  __syncwarp();
+  if (lane < C) {                              // lane j: column j of T by forward substitution, then of B T
+    float col[C];
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      const float beta = t < nc ? sigmoid_exact(p.b[(long)(start + t) * p.ldb + h]) : 0.f;
+      float v = t == lane ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) v = fmaf(-sA[warp][t * C + s], col[s], v);
+      col[t] = beta * v;
+      sT[warp][t * C + lane] = col[t];
+    }
+    float* M = tile + (3 * C + 1) * D;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      float m = 0.f;
+#pragma unroll
+      for (int s = 0; s <= t; ++s) m = fmaf(sB[warp][t * C + s], col[s], m);
+      M[t * C + lane] = col[t];
+      M[C * C + t * C + lane] = m;
+    }
+  }
+}
+// N sums held by every one of 2 O lanes: halve the sums a lane holds and the lanes that share them, step by step; once a
+// lane holds one, the last steps add.  Lane r of the group ends with the sums r N / (2 O) .. of the N
+template <int N, int O>
+__device__ __forceinline__ void reduce_scatter(float* a, int lane) {
+  if constexpr (O >= 1) {
+    if constexpr (N > 1) {
+      const bool up = (lane & O) != 0;
+#pragma unroll
+      for (int e = 0; e < N / 2; ++e) {
+        const float give = up ? a[e] : a[e + N / 2], keep = up ? a[e + N / 2] : a[e];
+        a[e] = keep + __shfl_xor_sync(0xffffffffu, give, O);
+      }
+      reduce_scatter<N / 2, O / 2>(a, lane);
+    } else {
+      a[0] += __shfl_xor_sync(0xffffffffu, a[0], O);
+      reduce_scatter<1, O / 2>(a, lane);
+    }
+  }
+}
+template <int P, int NC>
+__global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) {
+  // a column belongs to P lanes of one warp, NC neighbouring columns to the same lanes; a warp holds CW columns.  Chunk
+  // tiles are copied ahead (cp.async, two buffers); the rows of k~, q~, k^ are laid out LS_RS apart per lane (no bank conflicts)
+  constexpr int C = DC_C, D = P * LS_R, TILE = (3 * C + 1) * D + 2 * C * C, LD = P * LS_RS, ROWS = 3 * C + 1;
+  constexpr int NW = LS_THREADS / 32, CW = 32 / P * NC, PAIRS = (C * CW + 31) / 32, BUF = ROWS * LD + 2 * C * C;
+  constexpr int NV = 2 * C;                    // sums per column, reduced over P lanes: a lane ends with NL of them
+  constexpr int NL = P >= NV ? 1 : NV / P;
+  extern __shared__ __align__(16) float sm[];
+  float* red = sm + 2 * BUF + (threadIdx.x >> 5) * (CW * (NV + 2 * C));       // this warp's: sums [CW][2C], w [CW][C], u [CW][C]
+  float* wv = red + CW * NV;
+  float* us = wv + CW * C;
+  const int seq = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int start = p.seqs[2 * seq], rows = p.seqs[2 * seq + 1], n_chunks = (rows + C - 1) / C;
+  const int r = lane % P, cl = lane / P * NC;  // the lane's part of the rows; its first column within the warp
+  const int wcol = (blockIdx.z * NW + warp) * CW, col0 = wcol + cl;
+  const long head_floats = (long)LS_R * p.vdim * P;
+  float* st = p.state + (long)p.slot[start] * p.slot_stride + (long)h * head_floats;
+  const bool from_state = p.pos[start] > 0;
+  float S[NC][LS_R];
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
+#pragma unroll
+    for (int i = 0; i < LS_R; ++i) S[c][i] = (from_state && col0 + c < p.vdim) ? st[((long)i * p.vdim + col0 + c) * P + r] : 0.f;
+  const float* tiles = p.tiles + (first_chunk(p.seqs, seq) * p.H + h) * TILE;
+  auto fetch = [&](int c) {
+    const float* t = tiles + (long)c * p.H * TILE;
+    float* d = sm + (c & 1) * BUF;
+    for (int e = threadIdx.x; e < TILE / 4; e += LS_THREADS) {
+      const int f = e * 4, row = f / D, i = f % D;
+      float* to = row < ROWS ? d + row * LD + (i / LS_R) * LS_RS + i % LS_R : d + ROWS * LD + (f - ROWS * D);
+      const unsigned a = (unsigned)__cvta_generic_to_shared(to);
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(t + f) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float vn[PAIRS];                             // the values of the lane's (token, column) pairs, one chunk ahead
+  auto request_v = [&](int c) {
+#pragma unroll
+    for (int n = 0; n < PAIRS; ++n) {
+      const int e = lane + 32 * n, t = c * C + e / CW, col = wcol + e % CW;
+      vn[n] = (e < C * CW && t < rows && col < p.vdim) ? p.v[(long)(start + t) * p.ldv + (long)h * p.vdim + col] : 0.f;
+    }
+  };
+  fetch(0);
+  request_v(0);
+  for (int c = 0; c < n_chunks; ++c) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                           // this chunk's tile is here, and everyone has left the other buffer
+    if (c + 1 < n_chunks) fetch(c + 1);
+    const float* B = sm + (c & 1) * BUF;
+    float a[NC][NV];
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {             // rows 0 .. C-1: k~, C .. 2C-1: q~
+      const float* x = B + t * LD + r * LS_RS;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+      for (int j = 0; j < NC; ++j) {
+        float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < LS_R; i += 2) { s0 = fmaf(S[j][i], x_[i], s0); s1 = fmaf(S[j][i + 1], x_[i + 1], s1); }
+        a[j][t] = s0 + s1;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < NC; ++j) reduce_scatter<NV, P / 2>(a[j], lane);
+#pragma unroll
+    for (int j = 0; j < NC; ++j)
+#pragma unroll
+      for (int e = 0; e < NL; ++e) red[(cl + j) * NV + (P > NV ? r / (P / NV) : r * NL + e)] = a[j][e];
+    __syncwarp();
+    // a lane per (token, column): w = v - S^T k~
+#pragma unroll
+    for (int n = 0; n < PAIRS; ++n) {
+      const int e = lane + 32 * n, t = e / CW, cc = e % CW;
+      if (e < C * CW) wv[cc * C + t] = vn[n] - red[cc * NV + t];
+    }
+    __syncwarp();
+    const float* TT = B + ROWS * LD;
+#pragma unroll
+    for (int n = 0; n < PAIRS; ++n) {          // u_t = T_t . w,  o_t = S^T q~_t + (B T)_t . w
+      const int e = lane + 32 * n, t = e / CW, cc = e % CW;
+      if (e < C * CW) {
+        float u = 0.f, o = red[cc * NV + C + t];
+#pragma unroll
+        for (int s = 0; s < C; ++s) {
+          const float w = wv[cc * C + s];
+          u = fmaf(TT[t * C + s], w, u);
+          o = fmaf(TT[C * C + t * C + s], w, o);
+        }
+        us[cc * C + t] = u;
+        const int row = c * C + t;
+        if (row < rows && wcol + cc < p.vdim) p.out[(long)(start + row) * p.ldo + (long)h * p.vdim + wcol + cc] = o;
+      }
+    }
+    if (c + 1 < n_chunks) request_v(c + 1);
+    __syncwarp();
+    {
+      const float* x = B + 3 * C * LD + r * LS_RS;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+      for (int j = 0; j < NC; ++j)
+#pragma unroll
+        for (int i = 0; i < LS_R; ++i) S[j][i] *= x_[i];
+    }
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      const float* x = B + (2 * C + t) * LD + r * LS_RS;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+      for (int j = 0; j < NC; ++j) {
+        const float u = us[(cl + j) * C + t];
+#pragma unroll
+        for (int i = 0; i < LS_R; ++i) S[j][i] = fmaf(x_[i], u, S[j][i]);
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
+    if (col0 + c < p.vdim) {
+#pragma unroll
+      for (int i = 0; i < LS_R; ++i) st[((long)i * p.vdim + col0 + c) * P + r] = S[c][i];
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------
 // what follows a mixer's heads, written into a column range of the buffer the output projection reads:
 //   out[t][c] = scale * o[t][c] * [ rsqrt(mean over its group of `span` numbers + eps) * w[c mod w_len] ] * act(gate)
 // with the gate one number per element or per head, through a sigmoid or silu.  A warp per norm group.
@@ -947,54 +1304,38 @@ __global__ void head_post_kernel(HeadPostP p) {
 }
 
 // gated feed-forward activation with clamps: g = min(a, lim), u = clamp(b, -lim, lim),
-// y = g sigmoid(alpha (g + cubic g^3)) (u + up_off)
+// y = g sigmoid(alpha (g + cubic g^3)) (u + up_off), or, relu, y = max(g, 0) (u + up_off)
 // (lim = +inf, alpha = 1, cubic = 0, up_off = 0: the plain silu-gated unit; alpha = 2 sqrt(2 / pi), cubic = 0.044715: the
 // tanh form of gelu on the gate, since 0.5 (1 + tanh a) = sigmoid(2 a))
-__global__ void glu_clamp_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, float lim,
-                                 float alpha, float cubic, float up_off, float* __restrict__ Y, long ldy, int n) {
+__global__ void glu_clamp_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, GluP p,
+                                 float* __restrict__ Y, long ldy, int n) {
   const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x;
   if (i >= n) return;
-  const float g = fminf(G[(long)t * ldg + i], lim);
-  const float u = fminf(fmaxf(U[(long)t * ldu + i], -lim), lim);
-  Y[(long)t * ldy + i] = g * sigmoid_exact(alpha * glu_arg(g, cubic)) * (u + up_off);
+  Y[(long)t * ldy + i] = glu_unit(G[(long)t * ldg + i], U[(long)t * ldu + i], p);
 }
 // the same, four columns per thread (rows of whole, aligned 16-byte vectors)
-__global__ void glu_clamp4_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, float lim,
-                                  float alpha, float cubic, float up_off, float* __restrict__ Y, long ldy, int n) {
+__global__ void glu_clamp4_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, GluP p,
+                                  float* __restrict__ Y, long ldy, int n) {
   const int t = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
   if (i >= n) return;
   const float4 a = *reinterpret_cast<const float4*>(G + (long)t * ldg + i);
   const float4 b = *reinterpret_cast<const float4*>(U + (long)t * ldu + i);
-  const float gs[4] = {a.x, a.y, a.z, a.w}, us[4] = {b.x, b.y, b.z, b.w};
-  float y[4];
-#pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    const float g = fminf(gs[e], lim), u = fminf(fmaxf(us[e], -lim), lim);
-    y[e] = g * sigmoid_exact(alpha * glu_arg(g, cubic)) * (u + up_off);
-  }
-  *reinterpret_cast<float4*>(Y + (long)t * ldy + i) = make_float4(y[0], y[1], y[2], y[3]);
+  *reinterpret_cast<float4*>(Y + (long)t * ldy + i) =
+      make_float4(glu_unit(a.x, b.x, p), glu_unit(a.y, b.y, p), glu_unit(a.z, b.z, p), glu_unit(a.w, b.w, p));
 }
 
 // the same, written as the bf16 operand rows of the next tensor-core product (zero-padded to Kp columns)
-__global__ void glu_clamp_bf16_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, float lim,
-                                      float alpha, float cubic, float up_off, bf16* __restrict__ Y, int n, int Kp,
-                                      const int* __restrict__ live) {
+__global__ void glu_clamp_bf16_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, GluP p,
+                                      bf16* __restrict__ Y, int n, int Kp, const int* __restrict__ live) {
   const long t = blockIdx.x;
   const bool pad = live && live[t] < 0;          // a padding row of a sorted segment: zeros, its inputs are not read
-  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < Kp; i += blockDim.x * gridDim.y) {
-    float y = 0.f;
-    if (i < n && !pad) {
-      const float g = fminf(G[t * ldg + i], lim), u = fminf(fmaxf(U[t * ldu + i], -lim), lim);
-      y = g * sigmoid_exact(alpha * glu_arg(g, cubic)) * (u + up_off);
-    }
-    Y[t * Kp + i] = f2bf(y);
-  }
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < Kp; i += blockDim.x * gridDim.y)
+    Y[t * Kp + i] = f2bf((i < n && !pad) ? glu_unit(G[t * ldg + i], U[t * ldu + i], p) : 0.f);
 }
 
 // four columns per thread (rows of whole, aligned 16-byte vectors; n and Kp multiples of 4)
-__global__ void glu_clamp_bf16x4_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, float lim,
-                                        float alpha, float cubic, float up_off, bf16* __restrict__ Y, int n, int Kp,
-                                        const int* __restrict__ live) {
+__global__ void glu_clamp_bf16x4_kernel(const float* __restrict__ G, long ldg, const float* __restrict__ U, long ldu, GluP p,
+                                        bf16* __restrict__ Y, int n, int Kp, const int* __restrict__ live) {
   const long t = blockIdx.x;
   const bool pad = live && live[t] < 0;
   for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4; i < Kp; i += blockDim.x * gridDim.y * 4) {
@@ -1002,12 +1343,7 @@ __global__ void glu_clamp_bf16x4_kernel(const float* __restrict__ G, long ldg, c
     if (i < n && !pad) {
       const float4 a = *reinterpret_cast<const float4*>(G + t * ldg + i);
       const float4 b = *reinterpret_cast<const float4*>(U + t * ldu + i);
-      const float gs[4] = {a.x, a.y, a.z, a.w}, us[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float g = fminf(gs[e], lim), u = fminf(fmaxf(us[e], -lim), lim);
-        y[e] = g * sigmoid_exact(alpha * glu_arg(g, cubic)) * (u + up_off);
-      }
+      y[0] = glu_unit(a.x, b.x, p); y[1] = glu_unit(a.y, b.y, p); y[2] = glu_unit(a.z, b.z, p); y[3] = glu_unit(a.w, b.w, p);
     }
     const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
     uint2 pk;
@@ -1067,6 +1403,26 @@ __global__ void sink_softmax_bf16_kernel(const float* __restrict__ S, long lds, 
 }
 
 unsigned long long g_sink_attr_f32 = 0, g_sink_attr_bf16 = 0;
+
+// all chunks' tiles, then the walk.  Two columns per lane set when that still gives every SM a block.
+template <int P>
+int delta_chunks(const DeltaChunkP& p, int n_seq, int max_rows, cudaStream_t cs) {
+  static unsigned long long attr = 0;
+  constexpr int BUF = (3 * DC_C + 1) * P * LS_RS + 2 * DC_C * DC_C;
+  auto smem = [](int nc) { return (size_t)(2 * BUF + LS_THREADS / 32 * (32 / P * nc) * 4 * DC_C) * sizeof(float); };
+  if (first_use_on_device(&attr)) {
+    B200_CUDA(cudaFuncSetAttribute(delta_chunk_kernel<P, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem(1)));
+    B200_CUDA(cudaFuncSetAttribute(delta_chunk_kernel<P, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem(2)));
+  }
+  delta_chunk_prep_kernel<P><<<dim3(cdiv(max_rows, DC_C), cdiv(p.H, 4), n_seq), 128, 0, cs>>>(p);
+  B200_CHECK_LAUNCH();
+  const int cols = LS_THREADS / P;
+  const long two = (long)n_seq * p.H * cdiv(p.vdim, 2 * cols);
+  if (two >= 148) delta_chunk_kernel<P, 2><<<dim3(n_seq, p.H, cdiv(p.vdim, 2 * cols)), LS_THREADS, smem(2), cs>>>(p);
+  else delta_chunk_kernel<P, 1><<<dim3(n_seq, p.H, cdiv(p.vdim, cols)), LS_THREADS, smem(1), cs>>>(p);
+  B200_CHECK_LAUNCH();
+  return B200_OK;
+}
 
 }  // namespace
 }  // namespace b200
@@ -1129,6 +1485,27 @@ int b200_lm_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* 
   return B200_OK;
 }
 
+int b200_lm_head_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* V, long ldv, void* cache, int cache_bf16,
+                          long slot_stride, long tok_stride, const int* slot, const int* pos, const float* cs, int H, int G,
+                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int T,
+                          void* st) {
+  B200_REQUIRE(Q && K && V && cache && slot && pos && T > 0 && H > 0 && G > 0, "lm_head_qkv_post: bad argument");
+  B200_REQUIRE(rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || cs), "lm_head_qkv_post: rotated dims %d of %d", rot_dims, dim);
+  const int warps = T < 64 ? 2 : 8;            // few tokens: smaller blocks, so that the heads of a token spread over the SMs
+  const dim3 grid(T, cdiv(H + 2 * G, warps));
+  if (cache_bf16) {
+    HeadQkvP<bf16> p{Q, ldq, K, ldk, V, ldv, (bf16*)cache, slot_stride, tok_stride, slot, pos, (const float2*)cs, H, G, dim, vdim,
+                     rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps};
+    head_qkv_post_kernel<bf16><<<grid, warps * 32, 0, (cudaStream_t)st>>>(p);
+  } else {
+    HeadQkvP<float> p{Q, ldq, K, ldk, V, ldv, (float*)cache, slot_stride, tok_stride, slot, pos, (const float2*)cs, H, G, dim, vdim,
+                      rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps};
+    head_qkv_post_kernel<float><<<grid, warps * 32, 0, (cudaStream_t)st>>>(p);
+  }
+  B200_CHECK_LAUNCH();
+  return B200_OK;
+}
+
 int b200_lm_sink_attention(const float* q, long ldq, const void* cache, int cache_bf16, long slot_stride, long tok_stride,
                            const int* slot, const int* pos, float* out, long ldo, const void* sink, int H, int G,
                            int dim, int vdim, float scale, int chunk, int window, float bias_exp, int unit_sink, float* part,
@@ -1169,18 +1546,34 @@ int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, con
                          int H, int rep, int dim, int vdim, int act, float unit_eps, float q_scale,
                          const float* decay_const, const float* a, long lda, const void* A_log, const void* dt_bias,
                          const float* b, long ldb, int delta, int dt_in, const void* skip, const float* wraw, long ldwr,
-                         const void* bonus, float* prep, int part_len, int n_parts, float* part_scratch, int T, void* st) {
+                         const void* bonus, float* prep, int part_len, int n_parts, float* part_scratch, int max_rows, int T,
+                         void* st) {
   B200_REQUIRE(q && k && v && out && state && seqs && slot && pos && n_seq > 0 && H > 0 && rep > 0 && H % rep == 0,
                "lm_linear_state: bad argument");
   B200_REQUIRE(dim > 0 && dim <= 32 * LS_R && vdim > 0, "lm_linear_state: key size %d not supported (at most %d)", dim, 32 * LS_R);
   const bool chan = wraw != nullptr;
   B200_REQUIRE(chan || decay_const || (a && A_log && dt_bias), "lm_linear_state: a decay per head, or the inputs of a computed one");
-  B200_REQUIRE(!chan || (bonus && rep == 1 && !delta && !dt_in && !act && unit_eps == 0.f && !skip && !decay_const),
-               "lm_linear_state: a decay per key channel comes with a bonus and nothing else");
+  const bool chan_delta = chan && delta;
+  B200_REQUIRE(!chan || chan_delta || (bonus && rep == 1 && !dt_in && !act && unit_eps == 0.f && !skip && !decay_const),
+               "lm_linear_state: a decay per key channel comes with a bonus, or with the delta rule, and nothing else");
+  B200_REQUIRE(!chan_delta || (!bonus && !dt_in && !act && unit_eps > 0.f && !skip && !decay_const && A_log && dt_bias && b),
+               "lm_linear_state: the delta rule with a decay per key channel needs unit lengths, A_log, dt_bias and b");
   B200_REQUIRE(!dt_in || (!decay_const && !delta && !b), "lm_linear_state: the step size scales the input only in the plain form with a computed decay");
   StateP p{q, ldq, k, ldk, v, ldv, out, ldo, state, slot_stride, seqs, slot, pos, H, rep, dim, vdim, act, unit_eps, q_scale,
            nullptr, nullptr, nullptr, decay_const, a, lda, (const bf16*)A_log, (const bf16*)dt_bias, b, ldb, delta, dt_in, (const bf16*)skip, wraw, ldwr, (const bf16*)bonus, 0, 0, nullptr, nullptr};
   const cudaStream_t cs = (cudaStream_t)st;
+  if (chan_delta && prep) {      // a prompt step: chunk by chunk
+    B200_REQUIRE(max_rows > 0 && max_rows <= T, "lm_linear_state: the longest sequence of the step has %d of %d rows", max_rows, T);
+    B200_REQUIRE(n_seq <= 65535 && ((uintptr_t)prep & 15) == 0, "lm_linear_state: %d sequences in one step", n_seq);
+    DeltaChunkP d{q, ldq, k, ldk, v, ldv, out, ldo, state, slot_stride, seqs, slot, pos, H, rep, dim, vdim, unit_eps, q_scale,
+                  wraw, ldwr, (const bf16*)A_log, (const bf16*)dt_bias, b, ldb, prep};
+    if (dim <= LS_R) return delta_chunks<1>(d, n_seq, max_rows, cs);
+    if (dim <= 2 * LS_R) return delta_chunks<2>(d, n_seq, max_rows, cs);
+    if (dim <= 4 * LS_R) return delta_chunks<4>(d, n_seq, max_rows, cs);
+    if (dim <= 8 * LS_R) return delta_chunks<8>(d, n_seq, max_rows, cs);
+    if (dim <= 16 * LS_R) return delta_chunks<16>(d, n_seq, max_rows, cs);
+    return delta_chunks<32>(d, n_seq, max_rows, cs);
+  }
   if (prep) {     // scratch of T * (2 Hk dim + Hk + 2 H) floats: the per-token work runs first, over all tokens at once
     B200_REQUIRE(T > 0, "lm_linear_state: the prepared path needs the number of tokens");
     const int Hk = H / rep;
@@ -1209,7 +1602,8 @@ int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, con
       channel_state_kernel<PP, 2, false><<<pgrid, block, 0, cs>>>(p);                                            \
     } else if (chan && prep) {                                                                                   \
       channel_state_kernel<PP, 2, false><<<dim3(n_seq, H, cdiv(vdim, 2 * (LS_THREADS / PP))), block, 0, cs>>>(p); \
-    } else if (chan) linear_state_kernel<PP, false, true><<<grid, block, 0, cs>>>(p);                            \
+    } else if (chan_delta) linear_state_kernel<PP, true, true><<<grid, block, 0, cs>>>(p);                       \
+    else if (chan) linear_state_kernel<PP, false, true><<<grid, block, 0, cs>>>(p);                              \
     else if (delta) linear_state_kernel<PP, true, false><<<grid, block, 0, cs>>>(p);                             \
     else linear_state_kernel<PP, false, false><<<grid, block, 0, cs>>>(p);                                       \
   } while (0)
@@ -1256,23 +1650,25 @@ int b200_lm_head_post(const float* o, long ldi, const float* gate, long ldg, con
 }
 
 int b200_lm_glu_clamp(const float* G, long ldg, const float* U, long ldu, float limit, float alpha, float cubic, float up_off,
-                      float* Y, long ldy, int n, int T, void* st) {
+                      int relu, float* Y, long ldy, int n, int T, void* st) {
   B200_REQUIRE(G && U && Y && T > 0 && n > 0, "lm_glu_clamp: bad argument");
   const bool v4 = n % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && ldy % 4 == 0 &&
                   (((uintptr_t)G | (uintptr_t)U | (uintptr_t)Y) & 15) == 0;
-  if (v4 && T > 16) glu_clamp4_kernel<<<dim3(T, cdiv(n, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, limit, alpha, cubic, up_off, Y, ldy, n);
-  else glu_clamp_kernel<<<dim3(T, cdiv(n, 256)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, limit, alpha, cubic, up_off, Y, ldy, n);
+  const GluP p{limit, alpha, cubic, up_off, relu};
+  if (v4 && T > 16) glu_clamp4_kernel<<<dim3(T, cdiv(n, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, p, Y, ldy, n);
+  else glu_clamp_kernel<<<dim3(T, cdiv(n, 256)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, p, Y, ldy, n);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }
 
 int b200_lm_glu_clamp_bf16(const float* G, long ldg, const float* U, long ldu, float limit, float alpha, float cubic, float up_off,
-                           void* Y, int n, int Kp, const int* live, int T, void* st) {
+                           int relu, void* Y, int n, int Kp, const int* live, int T, void* st) {
   B200_REQUIRE(G && U && Y && T > 0 && n > 0 && Kp >= n, "lm_glu_clamp_bf16: bad argument");
   const bool v4 = n % 4 == 0 && Kp % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && (((uintptr_t)G | (uintptr_t)U) & 15) == 0 &&
                   ((uintptr_t)Y & 7) == 0;
-  if (v4) glu_clamp_bf16x4_kernel<<<dim3(T, cdiv(Kp, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, limit, alpha, cubic, up_off, (bf16*)Y, n, Kp, live);
-  else glu_clamp_bf16_kernel<<<dim3(T, cdiv(Kp, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, limit, alpha, cubic, up_off, (bf16*)Y, n, Kp, live);
+  const GluP p{limit, alpha, cubic, up_off, relu};
+  if (v4) glu_clamp_bf16x4_kernel<<<dim3(T, cdiv(Kp, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, p, (bf16*)Y, n, Kp, live);
+  else glu_clamp_bf16_kernel<<<dim3(T, cdiv(Kp, 1024)), 256, 0, (cudaStream_t)st>>>(G, ldg, U, ldu, p, (bf16*)Y, n, Kp, live);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }

@@ -322,10 +322,11 @@ class RunCache(_BaseCache):
     """What ONE run of a layer keeps for ONE request in a `StatePool` slot: the rows of its attention (if it has
     one) and its span of the slot's state (if it is recurrent), with the `KVCache` surface the generation loops use.
     A layer that runs several times (a repeated span of layers) has one of these per run.  A recurrent state cannot be
-    rolled back, so such a cache is not trimmable."""
+    rolled back, so such a cache is not trimmable.  `shared`: the rows are another layer's (read, never written)."""
 
     def __init__(self, pool: StatePool, row: int = 0, kv_layer: Optional[int] = None, kv_dim: int = 0,
-                 state_off: int = 0, state_len: int = 0):
+                 state_off: int = 0, state_len: int = 0, shared: bool = False):
+        self.shared = shared
         self._pool, self._row, self._layer = pool, row, kv_layer
         self._kv_dim, self._state_off, self._state_len = kv_dim, state_off, state_len
         self.offset = 0
@@ -374,7 +375,7 @@ class RunCache(_BaseCache):
     @property
     def nbytes(self):
         k = self.keys
-        return (0 if k is None else k.numel() * k.element_size()) + 4 * self._state_len
+        return (0 if k is None or self.shared else k.numel() * k.element_size()) + 4 * self._state_len
 
 
 def make_prompt_cache(model: Any, max_kv_size: Optional[int] = None) -> List[Any]:

@@ -40,6 +40,17 @@ on what the mixer reads:
                                                  erf-gelu experts, a shared expert)
   layer          ConvPreNormLayer: h = N1(x); h += conv(h); x += m * mixer(h); x += m * ff(N2(x))
 
+and, for layers that norm the SUM of a scaled stream and a branch (the sublayers read the stream itself):
+
+  mixers         NORMED_SUM_MIXERS["attention"]        -> GroupedAttention whose values are the projected keys: norms per head,
+                                                           rotation in pairs, frequencies scaled by wavelength, a window, one
+                                                           in the softmax's denominator
+                 NORMED_SUM_MIXERS["latent_attention"] -> LatentAttention without positions, a window, a gate per head, an
+                                                           earlier layer's latent if the configuration says so
+                 NORMED_SUM_MIXERS["channel_delta"]    -> ChannelDeltaRule (delta rule with a decay per key channel)
+  feed-forwards  NORMED_SUM_FEEDFORWARDS["dense"]      -> GatedDense with relu on the gate
+  layer          NormedSumLayer: x = LN(a * x + mixer(x)); x = LN(a * x + ff(x)), layer norms with a bias
+
 A block declares `manifest(prefix)` (packed name, shape) and `pack(prefix, checkpoint tensors, arena)`; the model
 packs all blocks into ONE device arena (the layout the other models of this package use).  `forward(ctx, x)`
 enqueues the block's kernels; `ctx` carries the per-token slot / position arrays of the step and the cache pool,
@@ -53,7 +64,8 @@ from typing import Dict, List, Optional
 import torch
 
 from .._native import B200Error as _B200Error
-from .layer_ops import ACT_GELU, ACT_TANH, EPI_GELU, EPI_RELU2, EPI_SOFTCAP, GELU_TANH_ALPHA, GELU_TANH_CUBIC, LayerOps
+from .layer_ops import (ACT_GELU, ACT_TANH, EPI_GELU, EPI_RELU2, EPI_SOFTCAP, GELU_TANH_ALPHA, GELU_TANH_CUBIC, WAVELENGTH,
+                        LayerOps)
 
 
 @dataclass
@@ -67,6 +79,8 @@ class StepCtx:
     _rope: Dict = field(default_factory=dict)
     _seq: Optional[tuple] = None
     carry: Dict = field(default_factory=dict)     # what one layer of the step leaves for later ones (rows of the step)
+    x_operand: Optional[torch.Tensor] = None      # bf16 operand rows of the residual stream, where the sublayers read the
+                                                  # stream itself and the norm that closed the last one wrote them
 
     def seq_tables(self):
         """(first (T,), seqs (G, 2), G): the sequences of the step for the mixers that walk them in order; without a
@@ -90,13 +104,16 @@ class LatentAttention:
     `kv_from = j`: no W_dkv, the rows that layer j cached are read instead (same rank and rotation).
     The rotation is on the first `rot_dims` of the rotated part, frequency base `rot_base`; its pairs are
     (i, i + rot_dims / 2) (`rotation="half"`) or (2i, 2i + 1) (`rotation="pairs"`); `rot.scaling` (factor, original,
-    fast, slow) rescales the frequencies by the YaRN rule and cos / sin by 0.1 ln(factor) + 1.
+    fast, slow) rescales the frequencies by the YaRN rule and cos / sin by 0.1 ln(factor) + 1.  Without `rot_dim` there is
+    no rotated part: the cache row is the latent alone.
     Without `q_rank` there is no query latent: q = W_q h.  `mask.size = w`: a query at position p sees the keys
-    p - w + 1 .. p.  `gated`: the heads' outputs are multiplied by sigmoid(W_g h) before W_o."""
+    p - w + 1 .. p.  `gated`: the heads' outputs are multiplied by sigmoid(W_g h) before W_o, one number per output
+    element ("element", or True) or per head ("head").  `split_weights`: in the tensor-core form of a long portion the
+    softmax's weights reach the value product as two bf16 parts (sixteen mantissa bits)."""
 
-    def __init__(self, index: int, cfg: dict, width: int, rotation: str = "half", gated: bool = False):
+    def __init__(self, index: int, cfg: dict, width: int, rotation: str = "half", gated=False, split_weights: bool = False):
         self.index, self.W = index, width
-        self.H, self.dim, self.rot_dim, self.vdim = cfg["heads"], cfg["dim"], cfg["rot_dim"], cfg["vdim"]
+        self.H, self.dim, self.rot_dim, self.vdim = cfg["heads"], cfg["dim"], int(cfg.get("rot_dim") or 0), cfg["vdim"]
         self.kv_rank, self.q_rank, self.scale = cfg["kv_rank"], int(cfg.get("q_rank") or 0), float(cfg["scale"])
         rot = cfg.get("rot") or {}
         self.rot_base, self.rot_dims = float(rot.get("base", 10000.0)), int(rot.get("dims", self.rot_dim))
@@ -105,7 +122,9 @@ class LatentAttention:
                                                 float(sc["slow"]))
         if rotation not in ("half", "pairs"):
             raise ValueError(f"layer {index}: rotation {rotation!r} (have 'half', 'pairs')")
-        self.pairs, self.gated = rotation == "pairs", bool(gated)
+        self.pairs, self.gated, self.gate_per_head = rotation == "pairs", bool(gated), gated == "head"
+        self.n_gate = 0 if not gated else (self.H if self.gate_per_head else self.H * self.vdim)
+        self.split_weights = bool(split_weights)
         self.window = int((cfg.get("mask") or {}).get("size", 0))
         self.kv_from: Optional[int] = cfg.get("kv_from")
         if not self.q_rank and self.kv_from is not None:
@@ -126,7 +145,7 @@ class LatentAttention:
     def manifest(self, p: str):
         # `down`: every product that reads the layer's input, stacked: [query latent, or the queries themselves |
         # kv latent, rotated key part | gate]
-        n_down = (self.q_rank or self.n_q) + (self.row_dim if self.own_kv else 0) + (self.H * self.vdim if self.gated else 0)
+        n_down = (self.q_rank or self.n_q) + (self.row_dim if self.own_kv else 0) + self.n_gate
         out = [(p + "down", (n_down, self.W))]
         if self.q_rank:
             out += [(p + "dq.norm", (self.q_rank,)), (p + "uq", (self.n_q, self.q_rank))]
@@ -147,7 +166,7 @@ class LatentAttention:
         if self.own_kv:
             out.update({p + "dkv": (self.row_dim, self.W), p + "dkv.norm": (self.kv_rank,)})
         if self.gated:
-            out[p + "g"] = (self.H * self.vdim, self.W)
+            out[p + "g"] = (self.n_gate, self.W)
         return out
 
     def pack(self, p: str, ck: Dict[str, torch.Tensor], view):
@@ -175,7 +194,7 @@ class LatentAttention:
         ops, w, T = ctx.ops, self.w, x.shape[0]
         H, dn, dr, r, dv = self.H, self.dim, self.rot_dim, self.kv_rank, self.vdim
         Dl = r + dr
-        D = ops.linear(x, w["down"])
+        D = ops.linear(x, w["down"], operand=ctx.x_operand)
         cache_layer = ctx.pool.buf[self.cache_index][..., :Dl]    # a pool row may be wider than this layer's
         cs = ctx.rope(self.rot_base, self.rot_dims, self.rot_scaling)
         if self.q_rank:
@@ -201,7 +220,8 @@ class LatentAttention:
                 heads_tc = False
         if not heads_tc:
             ops.gemm(q, w["ukT"], qa, M=T, N_=r, K=dn, xb=dn + dr, ldw=dn, wb=r * dn, yb=Dl, batch=H)
-        ops.rope_q(q, qa, cs, H, dn, dr, self.rot_dims, r, pairs=self.pairs)
+        if dr:
+            ops.rope_q(q, qa, cs, H, dn, dr, self.rot_dims, r, pairs=self.pairs)
         ol = ops.empty((T, H * r))
         segs = ctx.segments or []
         done = False
@@ -231,7 +251,7 @@ class LatentAttention:
         if not heads_tc:
             ops.gemm(ol, w["uv"], att, M=T, N_=dv, K=r, xb=r, ldw=r, wb=dv * r, yb=dv, batch=H)
         if self.gated:       # the gate reads the layer's input like the projections: the last columns of D
-            ops.head_post(att, att, dv=dv, gate=D[:, n_read:])
+            ops.head_post(att, att, dv=dv, gate=D[:, n_read:], gate_per_head=self.gate_per_head)
         return ops.linear(att, w["o"])
 
 
@@ -242,7 +262,8 @@ class LatentAttention:
         the weighted sum.  Queries are taken in chunks that bound the score buffer; with a window a chunk is about a
         window long and meets only the rows from its first query's first visible key on."""
         H, r, Dl = self.H, self.kv_rank, self.kv_rank + self.rot_dim
-        if not self.window:
+        parts = 2 if self.split_weights else 1
+        if not self.window and parts == 1:
             S = p0 + n
             Sp = (S + 63) // 64 * 64
             ct = ops.cache_transpose(rows, S, Sp, r)
@@ -256,20 +277,21 @@ class LatentAttention:
                 ops.masked_softmax_bf16(sc, pos[a:a + m], H, self.scale, P)
                 ops.tc_gemm(P, ct, ol[a:a + m].view(m * H, r), N_=r, K=Sp)
             return
-        step = max(128, min(self.window, (1 << 27) // (H * 2 * self.window)))
+        span = self.window or p0 + n
+        step = max(128, min(span, (1 << 27) // (H * 2 * span)))
         step = -(-n // -(-n // step))          # equal chunks: no short one at the end
         for a in range(0, n, step):
             m = min(step, n - a)
-            key0 = max(p0 + a - self.window + 1, 0)
+            key0 = max(p0 + a - self.window + 1, 0) if self.window else 0
             S = p0 + a + m - key0
             Sp = (S + 63) // 64 * 64
             ct = ops.cache_transpose(rows[key0:], S, Sp, r)
             qb = ops.to_bf16(qa[a:a + m].view(m * H, Dl), Dl)
             sc = ops.empty((m * H, S))
             ops.tc_gemm(qb, rows[key0:], sc, N_=S, K=Dl, ldw=rows.stride(0))
-            P = ops.empty((m * H, Sp), torch.bfloat16)
-            ops.sink_softmax_bf16(sc, pos[a:a + m], H, None, self.scale, 0, self.window, key0, P)
-            ops.tc_gemm(P, ct, ol[a:a + m].view(m * H, r), N_=r, K=Sp)
+            P = ops.empty((m * H, parts * Sp), torch.bfloat16)
+            ops.sink_softmax_bf16(sc, pos[a:a + m], H, None, self.scale, 0, self.window, key0, P, split=parts == 2)
+            ops.tc_gemm(P, ct, ol[a:a + m].view(m * H, r), N_=r, K=Sp, parts=parts)
 
 
 class ExpertMixture:
@@ -802,15 +824,16 @@ class GatedDense:
     """Gated feed-forward W_down (g sigmoid(alpha g) (u + offset)), g = min(W_gate n, limit), u = clamp(W_up n, +-limit);
     without a limit, alpha = 1 and offset = 0 it is the silu-gated unit W_down (silu(W_gate n) * W_up n).  Gate and up
     are one stacked product.  act = "gelu_tanh": the gate passes the tanh form of gelu instead,
-    g sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3)) = 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3)))."""
+    g sigmoid(2 sqrt(2 / pi) (g + 0.044715 g^3)) = 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3)));
+    act = "relu": max(g, 0)."""
 
     def __init__(self, index: int, cfg: dict, width: int, clamped: bool = False, alpha: float = 1.702, act: str = "silu"):
         self.index, self.W, self.ff = index, width, int(cfg["ff"])
         self.limit = float(cfg["limit"]) if clamped else float("inf")
         self.alpha, self.offset = (alpha, 1.0) if clamped else (1.0, 0.0)
-        if act not in ("silu", "gelu_tanh"):
-            raise ValueError(f"layer {index}: activation {act!r} (have 'silu', 'gelu_tanh')")
-        self.cubic = 0.0
+        if act not in ("silu", "gelu_tanh", "relu"):
+            raise ValueError(f"layer {index}: activation {act!r} (have 'silu', 'gelu_tanh', 'relu')")
+        self.cubic, self.relu = 0.0, act == "relu"
         if act == "gelu_tanh":
             self.alpha, self.cubic = GELU_TANH_ALPHA, GELU_TANH_CUBIC
         self.w: Dict[str, torch.Tensor] = {}
@@ -833,19 +856,20 @@ class GatedDense:
 
     def rows(self, ctx: StepCtx, x: torch.Tensor) -> torch.Tensor:
         ops = ctx.ops
-        D = ops.linear(x, self.w["gu"])
+        D = ops.linear(x, self.w["gu"], operand=ctx.x_operand)
         down = self.w["down"]
         if ops.tc_ok(x.shape[0], self.ff, down.stride(0)) and down.data_ptr() % 16 == 0:
             try:          # a prompt: the activation is written as the bf16 operand of the down product, in one pass
                 hb = ops.glu_clamp_bf16(D[:, :self.ff], D[:, self.ff:], self.limit, self.alpha, up_offset=self.offset,
-                                        cubic=self.cubic)
+                                        cubic=self.cubic, relu=self.relu)
                 y = ops.empty((x.shape[0], self.W))
                 ops.tc_gemm(hb, down, y, N_=self.W, K=self.ff, ldw=down.stride(0))
                 return y
             except _B200Error as e:
                 ops.tc_refused(e)
         hid = ops.empty((x.shape[0], self.ff))
-        ops.glu_clamp(D[:, :self.ff], D[:, self.ff:], self.limit, self.alpha, hid, up_offset=self.offset, cubic=self.cubic)
+        ops.glu_clamp(D[:, :self.ff], D[:, self.ff:], self.limit, self.alpha, hid, up_offset=self.offset, cubic=self.cubic,
+                      relu=self.relu)
         return ops.linear(hid, down)
 
     def forward(self, ctx: StepCtx, x: torch.Tensor) -> dict:
@@ -1029,8 +1053,12 @@ class ScaledPreNormLayer:
 class GroupedAttention:
     """Softmax attention with `heads` query heads over `kv_heads` key/value heads (query head h reads key/value head
     h // (heads / kv_heads)), q, k, v one stacked product of the mixer's input.  Optional, each by a parameter:
-      qk_norm     q and k are RMS-normed over their WHOLE projection (all heads at once) and weighted (`q.norm`, `k.norm`)
-      rot         rotate-half rotary on the first `rot.dims` numbers of every head, YaRN-scaled by `rot.scaling`
+      qk_norm     "whole" (or True): q and k are RMS-normed over their WHOLE projection (all heads at once) and weighted
+                  (`q.norm`, `k.norm`); "head": every head by itself, with one weight vector for all query (key) heads
+      rot         rotary on the first `rot.dims` numbers of every head, pairs (i, i + dims / 2) (rotation="half") or
+                  (2i, 2i + 1) ("pairs"), frequencies rescaled by `rot.scaling`: the YaRN rule (factor, original, fast,
+                  slow) or the rule by wavelength (factor, original, low, high)
+      v_from_k    the values are the keys as projected, before norm and rotation: no value projection
       v_unit      every value head is divided by its root mean square; the cache holds it so
       sink        "learned": a logit per head (`sink`) joins the softmax's denominator without a key or a value;
                   "unit": the denominator holds one more 1 (a sink logit of zero)
@@ -1040,8 +1068,8 @@ class GroupedAttention:
       v_mix       the model marks the first mixing layer (`v_role = "first"`: its cached values are also kept for the
                   step) and the later ones (`"blend"`: v <- (1 - lam) v + lam v_first, lam = `vmix`, after the value norm)."""
 
-    def __init__(self, index: int, cfg: dict, width: int, qk_norm: bool = False, v_unit: bool = False,
-                 sink: Optional[str] = None, bias_exp: float = 0.0):
+    def __init__(self, index: int, cfg: dict, width: int, qk_norm=False, v_unit: bool = False,
+                 sink: Optional[str] = None, bias_exp: float = 0.0, rotation: str = "half", v_from_k: bool = False):
         self.index, self.W = index, width
         self.H, self.dim = int(cfg["heads"]), int(cfg["dim"])
         self.G, self.vdim = int(cfg.get("kv_heads", self.H)), int(cfg.get("vdim", self.dim))
@@ -1051,7 +1079,10 @@ class GroupedAttention:
         rot = cfg.get("rot") or {}
         self.rot_base, self.rot_dims = float(rot.get("base", 10000.0)), int(rot.get("dims", 0))
         sc = rot.get("scaling")
-        self.rot_scaling = None if not sc else (float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"]))
+        if sc and "low" in sc:
+            self.rot_scaling = (WAVELENGTH, float(sc["factor"]), float(sc["original"]), float(sc["low"]), float(sc["high"]))
+        else:
+            self.rot_scaling = None if not sc else (float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"]))
         if self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError(f"layer {index}: {self.rot_dims} rotated numbers in heads of {self.dim}")
         self.window = int((cfg.get("mask") or {}).get("size", 0))
@@ -1059,18 +1090,29 @@ class GroupedAttention:
         self.q_temp = None if not qt else (float(qt["coef"]), int(qt["every"]))
         if sink not in (None, "learned", "unit"):
             raise ValueError(f"layer {index}: sink {sink!r} (have None, 'learned', 'unit')")
+        if rotation not in ("half", "pairs") or qk_norm not in (False, True, "whole", "head"):
+            raise ValueError(f"layer {index}: rotation {rotation!r} (have 'half', 'pairs'), query/key norm {qk_norm!r}")
         self.qk_norm, self.v_unit, self.sink, self.bias_exp = bool(qk_norm), bool(v_unit), sink, float(bias_exp)
+        self.head_norm, self.pairs, self.v_from_k = qk_norm == "head", rotation == "pairs", bool(v_from_k)
+        self.per_head = self.head_norm or self.pairs      # the step between projection and cache is the per-head one
         self.v_mix = bool(cfg.get("v_mix"))
         self.v_role: Optional[str] = None      # set by the model: "first" / "blend"
+        if self.per_head and (self.v_unit or self.q_temp or self.v_mix or (qk_norm and not self.head_norm)):
+            raise ValueError(f"layer {index}: norms or rotation per head do not go with unit values, value mixing, a query "
+                             f"temperature or norms over the whole projection")
+        if self.v_from_k and (self.vdim != self.dim or self.v_mix):
+            raise ValueError(f"layer {index}: values that are the keys have the keys' size ({self.vdim} and {self.dim})")
         self.n_q, self.n_k, self.n_v = self.H * self.dim, self.G * self.dim, self.G * self.vdim
         self.kv_dim, self.state_floats = self.n_k + self.n_v, 0
         self.cache_index, self.state_off = -1, 0
         self.w: Dict[str, torch.Tensor] = {}
 
     def manifest(self, p: str):
-        out = [(p + "qkv", (self.n_q + self.n_k + self.n_v, self.W)), (p + "o", (self.W, self.H * self.vdim))]
+        out = [(p + "qkv", (self.n_q + self.n_k + (0 if self.v_from_k else self.n_v), self.W)),
+               (p + "o", (self.W, self.H * self.vdim))]
         if self.qk_norm:
-            out += [(p + "q.norm", (self.n_q,)), (p + "k.norm", (self.n_k,))]
+            out += [(p + "q.norm", (self.dim if self.head_norm else self.n_q,)),
+                    (p + "k.norm", (self.dim if self.head_norm else self.n_k,))]
         if self.sink == "learned":
             out.append((p + "sink", (self.H,)))
         if self.v_mix:
@@ -1078,10 +1120,10 @@ class GroupedAttention:
         return out
 
     def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
-        out = {p + "q": (self.n_q, self.W), p + "k": (self.n_k, self.W), p + "v": (self.n_v, self.W),
-               p + "o": (self.W, self.H * self.vdim)}
-        if self.qk_norm:
-            out.update({p + "q.norm": (self.n_q,), p + "k.norm": (self.n_k,)})
+        out = {p + "q": (self.n_q, self.W), p + "k": (self.n_k, self.W), p + "o": (self.W, self.H * self.vdim)}
+        if not self.v_from_k:
+            out[p + "v"] = (self.n_v, self.W)
+        out.update({n: s for n, s in self.manifest(p) if n in (p + "q.norm", p + "k.norm")})
         if self.sink == "learned":
             out[p + "sink"] = (self.H,)
         if self.v_mix:
@@ -1092,7 +1134,8 @@ class GroupedAttention:
         qkv = view(p + "qkv")
         qkv[:self.n_q].copy_(ck[p + "q"])
         qkv[self.n_q:self.n_q + self.n_k].copy_(ck[p + "k"])
-        qkv[self.n_q + self.n_k:].copy_(ck[p + "v"])
+        if not self.v_from_k:
+            qkv[self.n_q + self.n_k:].copy_(ck[p + "v"])
         for n, shape in self.manifest(p)[1:]:
             view(n).copy_(ck[n].reshape(shape))
         self.bind(p, view)
@@ -1103,18 +1146,23 @@ class GroupedAttention:
     def forward(self, ctx: StepCtx, h: torch.Tensor) -> torch.Tensor:
         ops, w, T = ctx.ops, self.w, h.shape[0]
         nq, nk, nv = self.n_q, self.n_k, self.n_v
-        D = ops.linear(h, w["qkv"])
-        q, k, v = D[:, :nq], D[:, nq:nq + nk], D[:, nq + nk:]
+        D = ops.linear(h, w["qkv"], operand=ctx.x_operand)
+        q, k = D[:, :nq], D[:, nq:nq + nk]
+        v = k if self.v_from_k else D[:, nq + nk:]
         rows = ctx.pool.buf[self.cache_index][..., :self.kv_dim]
+        cs = ctx.rope(self.rot_base, self.rot_dims, self.rot_scaling)
         v_first = keep = None
         if self.v_role == "first":
             keep = ctx.carry["v_first"] = ops.empty((T, nv))
         elif self.v_role == "blend":
             v_first = ctx.carry["v_first"]
-        ops.qkv_post(q, k, v, rows, ctx.slot, ctx.pos, ctx.rope(self.rot_base, self.rot_dims, self.rot_scaling), self.H, self.G,
-                     self.dim, self.vdim, self.rot_dims, q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps,
-                     v_unit=self.v_unit, q_temp=self.q_temp, vmix=w["vmix"] if v_first is not None else None,
-                     v_first=v_first, v_keep=keep)
+        if self.per_head:
+            ops.head_qkv_post(q, k, v, rows, ctx.slot, ctx.pos, cs, self.H, self.G, self.dim, self.vdim, self.rot_dims,
+                              q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps, pairs=self.pairs)
+        else:
+            ops.qkv_post(q, k, v, rows, ctx.slot, ctx.pos, cs, self.H, self.G, self.dim, self.vdim, self.rot_dims,
+                         q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps, v_unit=self.v_unit, q_temp=self.q_temp,
+                         vmix=w["vmix"] if v_first is not None else None, v_first=v_first, v_keep=keep)
         o = ops.empty((T, self.H * self.vdim))
         segs = ctx.segments or []
         done = False
@@ -1486,20 +1534,179 @@ class ConvPreNormLayer:
         return n
 
 
-def assign_cache_layers(layers: List[PostNormLayer]) -> int:
-    """number the layers that cache rows of their own; a borrowing layer gets its source's number"""
+# ----------------------------------------------------------------------------------------------------------------
+# Layers that norm the sum.  A mixer has `forward(ctx, x) -> rows (T, width)`, `kv_dim` / `cache_index` and
+# `state_floats` / `state_off` like the mixers of a ScaledPreNormLayer, and may take the bf16 operand rows of x from
+# `ctx.x_operand`; a feed-forward has `rows(ctx, x) -> rows (T, width)`.
+class ChannelDeltaRule:
+    """Gated delta rule with a decay per head and key channel: per head a (dim, vdim) state, fp32 in the slot, zero at
+    position 0, with  S <- diag(g) S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q.
+    q, k (`kv_heads` heads, shared by heads / kv_heads value heads) and v pass a short causal convolution per channel
+    (`conv` taps, no bias; the slot keeps the last taps - 1 inputs) and silu; q, k are then scaled to unit length per head
+    (q also by dim^-1/2); beta = sigmoid(W_b x); g = exp(-exp(A_log_h) softplus(W_a2 W_a1 x + dt_bias)), heads x dim;
+    every head's o is RMS-normed over vdim, times `norm` (vdim numbers, shared by the heads), times
+    sigmoid(W_g2 W_g1 x), then W_o.  The ranks of the two low-rank projections are the first sizes of their `a1` / `g1`
+    tensors (`a_rank` / `g_rank` in the configuration override them)."""
+    LOW_RANK = ("a", "g")
+
+    def __init__(self, index: int, cfg: dict, width: int, unit_eps: float = 1e-6):
+        self.index, self.W, self.unit_eps = index, width, unit_eps
+        self.H, self.dim, self.taps = int(cfg["heads"]), int(cfg["dim"]), int(cfg.get("conv") or 1)
+        self.G, self.vdim = int(cfg.get("kv_heads", self.H)), int(cfg.get("vdim", self.dim))
+        if self.H % self.G:
+            raise ValueError(f"layer {index}: {self.H} value heads do not divide over {self.G} query/key heads")
+        self.rank = {s: int(cfg.get(s + "_rank", 0)) for s in self.LOW_RANK}     # 0: taken from the checkpoint
+        self.n_qk, self.n_v, self.n_a = self.G * self.dim, self.H * self.vdim, self.H * self.dim
+        self.n_conv = 2 * self.n_qk + self.n_v
+        self.kv_dim = 0
+        self.conv_floats = max(self.taps - 1, 0) * self.n_conv
+        self.state_floats = self.conv_floats + state_floats(self.H, self.dim, self.vdim)
+        self.cache_index, self.state_off = -1, 0
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def set_rank(self, which: str, rank: int):
+        self.rank[which] = int(rank)
+
+    @property
+    def paired(self) -> bool:
+        """both second low-rank projections have the same shape: they are packed together and run as one batched product"""
+        return self.rank["a"] == self.rank["g"] and self.n_a == self.n_v
+
+    def _in(self):
+        """(name, rows) of everything that reads x, stacked in this order into one product"""
+        return [("q", self.n_qk), ("k", self.n_qk), ("v", self.n_v), ("a1", self.rank["a"]), ("g1", self.rank["g"]), ("b", self.H)]
+
+    def manifest(self, p: str):
+        n_in = (sum(n for _, n in self._in()) + 7) // 8 * 8          # whole vectors per row; the rows beyond are zeros
+        low = [(p + "ag2", (2, self.n_a, self.rank["a"]))] if self.paired else \
+            [(p + "a2", (self.n_a, self.rank["a"])), (p + "g2", (self.n_v, self.rank["g"]))]
+        return [(p + "in", (n_in, self.W)), (p + "conv", (self.n_conv, self.taps)), (p + "A_log", (self.H,)),
+                (p + "dt_bias", (self.n_a,)), (p + "norm", (self.vdim,)), (p + "o", (self.W, self.n_v))] + low
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        out = {p + s: (n, self.W) for s, n in self._in()}
+        out.update({p + s + ".conv": (n, self.taps) for s, n in self._in()[:3]})
+        out.update({p + "a2": (self.n_a, self.rank["a"]), p + "g2": (self.n_v, self.rank["g"]), p + "A_log": (self.H,),
+                    p + "dt_bias": (self.n_a,), p + "norm": (self.vdim,), p + "o": (self.W, self.n_v)})
+        return out
+
+    def pack(self, p: str, ck, view):
+        w_in, conv, r = view(p + "in"), view(p + "conv"), 0
+        for s, n in self._in():
+            w_in[r:r + n].copy_(ck[p + s])
+            if r + n <= self.n_conv:
+                conv[r:r + n].copy_(ck[p + s + ".conv"])
+            r += n
+        w_in[r:].zero_()
+        for i, s in enumerate(("a2", "g2")):
+            (view(p + "ag2")[i] if self.paired else view(p + s)).copy_(ck[p + s])
+        for s in ("A_log", "dt_bias", "norm", "o"):
+            view(p + s).copy_(ck[p + s])
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n[len(p):]: view(n) for n, _ in self.manifest(p)}
+
+    def forward(self, ctx: StepCtx, x: torch.Tensor) -> torch.Tensor:
+        ops, w, T = ctx.ops, self.w, x.shape[0]
+        n, nc, ra, rg = self.n_qk, self.n_conv, self.rank["a"], self.rank["g"]
+        st, off = ctx.pool.state, self.state_off
+        D = ops.linear(x, w["in"], operand=ctx.x_operand)
+        c = ops.short_conv(D[:, :nc], w["conv"], st[:, off:off + self.conv_floats], ctx, act=True)
+        low_a, low_g, beta = D[:, nc:nc + ra], D[:, nc + ra:nc + ra + rg], D[:, nc + ra + rg:]
+        if self.paired and not ops.tc_ok(T, ra):     # few rows: ONE launch over both (input, weight) pairs
+            both = ops.empty((2, T, self.n_a))
+            ops.gemm(low_a, w["ag2"], both, M=T, N_=self.n_a, K=ra, ldx=D.stride(0), xb=ra, ldw=ra, wb=self.n_a * ra,
+                     ldy=self.n_a, yb=T * self.n_a, batch=2)
+            logit, gate = both[0], both[1]
+        else:
+            a2, g2 = (w["ag2"][0], w["ag2"][1]) if self.paired else (w["a2"], w["g2"])
+            logit, gate = ops.linear(low_a, a2), ops.linear(low_g, g2)
+        o = ops.empty((T, self.n_v))
+        ops.linear_state(c[:, :n], c[:, n:2 * n], c[:, 2 * n:], o, st[:, off + self.conv_floats:off + self.state_floats], ctx,
+                         H=self.H, rep=self.H // self.G, dim=self.dim, vdim=self.vdim, unit_eps=self.unit_eps,
+                         q_scale=float(self.dim) ** -0.5, A_log=w["A_log"], dt_bias=w["dt_bias"], b=beta, delta=True,
+                         decay_logits=logit)
+        ops.head_post(o, o, dv=self.vdim, gate=gate, w=w["norm"], eps=ctx.eps, span=self.vdim)
+        return ops.linear(o, w["o"])
+
+
+NORMED_SUM_MIXERS = {"attention": lambda i, c, w: GroupedAttention(i, c, w, qk_norm="head", sink="unit", rotation="pairs",
+                                                                   v_from_k=True),
+                     "latent_attention": lambda i, c, w: LatentAttention(i, c, w, gated="head", split_weights=True),
+                     "channel_delta": ChannelDeltaRule}
+NORMED_SUM_FEEDFORWARDS = {"dense": lambda i, c, w: GatedDense(i, c, w, act="relu")}
+
+
+class NormedSumLayer:
+    """x <- N1(a x + mixer(x));  x <- N2(a x + ff(x)),  N(y) = (y - mean) / sqrt(var + eps) * w + b, a one number of the
+    model; the sublayers read x itself.  The residual stream, both sums and the norms are fp32; sum and norm are one launch,
+    which in a prompt also writes the bf16 operand rows that the next sublayer's first product reads."""
+
+    def __init__(self, index: int, cfg: dict, width: int, alpha: float = 1.0):
+        self.index, self.W, self.alpha = index, width, float(alpha)
+        if cfg["type"] not in NORMED_SUM_MIXERS:
+            raise ValueError(f"layer {index}: unknown mixer type {cfg['type']!r} (have {sorted(NORMED_SUM_MIXERS)})")
+        self.mixer = NORMED_SUM_MIXERS[cfg["type"]](index, cfg["mixer"], width)
+        f = cfg.get("mlp")
+        if f is not None and f.get("kind") not in NORMED_SUM_FEEDFORWARDS:
+            raise ValueError(f"layer {index}: unknown feed-forward kind {f.get('kind')!r} (have {sorted(NORMED_SUM_FEEDFORWARDS)})")
+        self.ff = None if f is None else NORMED_SUM_FEEDFORWARDS[f["kind"]](index, f, width)
+        self.kv_dim, self.state_floats = self.mixer.kv_dim, self.mixer.state_floats
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def _own(self):
+        return ["norm1", "norm1.b"] + (["norm2", "norm2.b"] if self.ff is not None else [])
+
+    def manifest(self, p: str):
+        out = [(p + n, (self.W,)) for n in self._own()] + self.mixer.manifest(p + "mix.")
+        return out + (self.ff.manifest(p + "mlp.") if self.ff is not None else [])
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        out = {p + n: (self.W,) for n in self._own()}
+        out.update(self.mixer.checkpoint_tensors(p + "mix."))
+        if self.ff is not None:
+            out.update(self.ff.checkpoint_tensors(p + "mlp."))
+        return out
+
+    def pack(self, p: str, ck, view):
+        for n in self._own():
+            view(p + n).copy_(ck[p + n])
+        self.mixer.pack(p + "mix.", ck, view)
+        if self.ff is not None:
+            self.ff.pack(p + "mlp.", ck, view)
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n: view(p + n) for n in self._own()}
+        self.mixer.bind(p + "mix.", view)
+        if self.ff is not None:
+            self.ff.bind(p + "mlp.", view)
+
+    def forward(self, ctx: StepCtx, x: torch.Tensor):
+        self._close(ctx, x, self.mixer.forward(ctx, x), "norm1")
+        if self.ff is not None:
+            self._close(ctx, x, self.ff.rows(ctx, x), "norm2")
+
+    def _close(self, ctx: StepCtx, x, y, norm: str):
+        ctx.x_operand = ctx.ops.sum_norm_rows(y, x, self.w[norm], self.w[norm + ".b"], ctx.eps, keep=self.alpha, center=True)
+
+
+def assign_cache_layers(layers: List) -> int:
+    """number the layers that cache rows of their own; a layer that borrows a latent gets its source's number"""
     n = 0
     for L in layers:
-        if L.mixer.own_kv:
-            L.mixer.cache_index = n
+        m = L.mixer
+        if m.kv_dim and getattr(m, "own_kv", True):
+            m.cache_index = n
             n += 1
     for L in layers:
         m = L.mixer
-        if not m.own_kv:
+        if not getattr(m, "own_kv", True):
             if not 0 <= m.kv_from < m.index:
                 raise ValueError(f"layer {m.index} borrows the latent of layer {m.kv_from}, which does not run before it")
             src = layers[m.kv_from].mixer
-            if not src.own_kv or (src.kv_rank, src.rot_dim, src.rot_base, src.rot_dims) != \
+            if not isinstance(src, LatentAttention) or not src.own_kv or (src.kv_rank, src.rot_dim, src.rot_base, src.rot_dims) != \
                     (m.kv_rank, m.rot_dim, m.rot_base, m.rot_dims):
                 raise ValueError(f"layer {m.index} borrows the latent of layer {m.kv_from}, which does not fit")
             m.cache_index = src.cache_index

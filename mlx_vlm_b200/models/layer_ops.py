@@ -18,6 +18,7 @@ from .. import _native as N
 EPI_NONE, EPI_RELU2, EPI_SOFTCAP, EPI_ADD, EPI_SCALE, EPI_GELU = 0, 1, 2, 3, 4, 5
 ACT_NONE, ACT_RELU2, ACT_GELU, ACT_TANH = 0, 1, 2, 3     # activation codes of `to_bf16` (gelu: the exact, erf form)
 GELU_TANH_ALPHA, GELU_TANH_CUBIC = 1.5957691216057308, 0.044715     # z sigmoid(alpha (z + cubic z^3)) = the tanh form of gelu
+WAVELENGTH = "wavelength"     # first entry of a frequency scaling by wavelength (a YaRN scaling is four numbers)
 SM_COUNT = 148
 TC_MIN_ROWS = 128     # from this many rows on, a product of the bf16 serving mode runs on the tcgen05 GEMM
 WT_F32 = 3            # gemm_wt output mode: fp32 rows
@@ -89,12 +90,20 @@ class LayerOps:
         Extension of Large Language Models"): with d(t) = dims ln(original / (2 pi t)) / (2 ln base) the index at
         which a frequency makes t turns over `original` positions, lo = max(floor d(fast), 0),
         hi = min(ceil d(slow), dims - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency is
-        f_i (1 - r_i) + (f_i / factor) r_i."""
+        f_i (1 - r_i) + (f_i / factor) r_i.
+        scaling = ("wavelength", factor, original, low, high), the rule of Llama 3.1: with n_i = original f_i / (2 pi)
+        the turns over `original` positions, f_i stays where n_i > high, becomes f_i / factor where n_i < low, and in
+        between is blended with r_i = (high - n_i) / (high - low) as above."""
         key = (float(base), int(dims), scaling)
         if key not in self._inv_freq:
             half = dims // 2
             f = np.power(np.float64(base), -2.0 * np.arange(half, dtype=np.float64) / dims)
-            if scaling is not None:
+            if scaling is not None and scaling[0] == WAVELENGTH:
+                factor, original, low, high = (float(v) for v in scaling[1:])
+                turns = original * f / (2.0 * np.pi)
+                ramp = np.clip((high - turns) / max(high - low, 1e-300), 0.0, 1.0)
+                f = f / factor * ramp + f * (1.0 - ramp)
+            elif scaling is not None:
                 factor, original, fast, slow = (float(v) for v in scaling)
 
                 def index(turns):
@@ -108,8 +117,8 @@ class LayerOps:
 
     @staticmethod
     def rope_amplitude(scaling: Optional[tuple]) -> float:
-        """what a frequency scaling multiplies cos and sin by: 0.1 ln(factor) + 1"""
-        return 1.0 if scaling is None else 0.1 * float(np.log(float(scaling[0]))) + 1.0
+        """what a frequency scaling multiplies cos and sin by: 0.1 ln(factor) + 1 (YaRN), 1 (by wavelength)"""
+        return 1.0 if scaling is None or scaling[0] == WAVELENGTH else 0.1 * float(np.log(float(scaling[0]))) + 1.0
 
     def rope_table(self, pos: torch.Tensor, base: float, dims: int, scaling: Optional[tuple] = None) -> torch.Tensor:
         T, half = pos.shape[0], dims // 2
@@ -122,14 +131,16 @@ class LayerOps:
 
     def norm_rows(self, y: torch.Tensor, w: torch.Tensor, eps: float, x: torch.Tensor, *, w_offset: float = 0.0,
                   add: bool = False, combine: Optional[torch.Tensor] = None, top: int = 0,
-                  rows: Optional[torch.Tensor] = None, center: bool = False, groups: int = 1):
-        """x (T, N) = or += rmsnorm(y rows) * (w_offset + w); `combine` (T, top): y holds `top` rows per token;
-        center: the mean of the row is taken off first (a layer norm without bias); groups: the row is that many equal
+                  rows: Optional[torch.Tensor] = None, center: bool = False, groups: int = 1,
+                  bias: Optional[torch.Tensor] = None):
+        """x (T, N) = or += rmsnorm(y rows) * (w_offset + w) [+ bias]; `combine` (T, top): y holds `top` rows per token;
+        center: the mean of the row is taken off first (a layer norm); groups: the row is that many equal
         consecutive parts, each divided by its own root mean square"""
         T, n = x.shape
         self._ok(self.lib.b200_lm_norm_rows(y.data_ptr(), y.stride(0), N.ptr(combine), int(top), w.data_ptr(),
                                             float(w_offset), float(eps), x.data_ptr(), x.stride(0), int(add),
-                                            N.ptr(rows), int(center), int(groups), T, n, self.s), "lm_norm_rows")
+                                            N.ptr(rows), int(center), int(groups), N.ptr(bias), T, n, self.s),
+                 "lm_norm_rows")
 
     def residual_rows(self, y: torch.Tensor, x: torch.Tensor, ls: Optional[torch.Tensor] = None, *,
                       combine: Optional[torch.Tensor] = None, top: int = 0, shared: Optional[torch.Tensor] = None,
@@ -154,8 +165,21 @@ class LayerOps:
             y.data_ptr(), y.stride(0), N.ptr(combine), int(top), N.ptr(shared), shared.stride(0) if shared is not None else 0,
             N.ptr(shared_gate), shared_gate.stride(0) if shared_gate is not None else 0, N.ptr(ls), x.data_ptr(), x.stride(0),
             w.data_ptr(), float(w_offset), float(eps), int(center), out.data_ptr(), out.stride(0), int(groups), float(mult),
-            T, n, self.s),
+            0, 1.0, 0, 0, T, n, self.s),
             "lm_residual_norm_rows")
+
+    def sum_norm_rows(self, y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], eps: float, *,
+                      keep: float = 1.0, center: bool = False) -> Optional[torch.Tensor]:
+        """x (T, N) = norm(keep * x + y) * w + bias in place (a stream that is normed after every sum; center: a layer
+        norm).  For a step whose products run on the tensor cores the result is also written as their bf16 operand rows
+        (T, ceil64(N)), returned"""
+        T, n = x.shape
+        xb = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16) if self.tc_ok(T, n) else None
+        self._ok(self.lib.b200_lm_residual_norm_rows(
+            y.data_ptr(), y.stride(0), 0, 0, 0, 0, 0, 0, 0, x.data_ptr(), x.stride(0), w.data_ptr(), 0.0, float(eps),
+            int(center), x.data_ptr(), x.stride(0), 1, 1.0, N.ptr(bias), float(keep), N.ptr(xb),
+            xb.stride(0) if xb is not None else 0, T, n, self.s), "lm_residual_norm_rows")
+        return xb
 
     def latent_post(self, D, wq, wkv, eps, cq, cache_layer, slot, pos, cs, q_rank, kv_rank, rot_dim, rot_dims,
                     pairs: bool = False):
@@ -322,12 +346,13 @@ class LayerOps:
         return out
 
     def linear(self, X: torch.Tensor, W: torch.Tensor, bias=None, epi=EPI_NONE, epi_param=0.0,
-               out: Optional[torch.Tensor] = None, add: bool = False, exact_x: bool = False) -> torch.Tensor:
+               out: Optional[torch.Tensor] = None, add: bool = False, exact_x: bool = False,
+               operand: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Y = epi(X . W^T + bias).  X and W may be column ranges of wider rows (their row pitch is taken from the
         tensors).  out: the rows to write (else fresh ones); add: the product is added to what `out` holds;
         exact_x: the rows of X are not rounded to one bf16 part in the serving mode (small products whose result
         decides something: a router): fp32 rows on the row kernels, or, for a long step, [hi | lo] halves on the
-        tensor cores."""
+        tensor cores; operand: the bf16 operand rows of X, if a previous launch already wrote them."""
         (T, K), n = X.shape, W.shape[0]
         Y = self.empty((T, n)) if out is None else out
         ldw = W.stride(0) if n > 1 else K
@@ -339,7 +364,8 @@ class LayerOps:
                 if exact_x:
                     self.tc_gemm(self.to_split(X, K), W, Y, N_=n, K=K, ldw=ldw, bias=bias, res=Y if add else None, parts=2)
                 else:
-                    self.tc_gemm(self.to_bf16(X, K), W, Y, N_=n, K=K, ldw=ldw, bias=bias, res=Y if add else None)
+                    self.tc_gemm(self.to_bf16(X, K) if operand is None else operand, W, Y, N_=n, K=K, ldw=ldw, bias=bias,
+                                 res=Y if add else None)
                 return Y
             except N.B200Error as e:
                 self.tc_refused(e)
@@ -408,6 +434,16 @@ class LayerOps:
                                            N.ptr(v_keep), v_keep.stride(0) if v_keep is not None else 0, Q.shape[0], self.s),
                  "lm_qkv_post")
 
+    def head_qkv_post(self, Q, K, V, cache_layer, slot, pos, cs, H, G, dim, vdim, rot_dims, *, q_norm=None, k_norm=None,
+                      eps: float = 0.0, pairs: bool = False):
+        """`qkv_post` with everything per head: q_norm / k_norm (dim,): RMS norm of every head times ONE weight for all
+        heads; pairs: the rotation pairs (2i, 2i + 1).  V may be K itself"""
+        self._ok(self.lib.b200_lm_head_qkv_post(
+            Q.data_ptr(), Q.stride(0), K.data_ptr(), K.stride(0), V.data_ptr(), V.stride(0), cache_layer.data_ptr(),
+            int(cache_layer.dtype == torch.bfloat16), cache_layer.stride(0), cache_layer.stride(1), slot.data_ptr(),
+            pos.data_ptr(), cs.data_ptr(), H, G, dim, vdim, rot_dims, int(pairs), N.ptr(q_norm), N.ptr(k_norm), float(eps),
+            Q.shape[0], self.s), "lm_head_qkv_post")
+
     def sink_attention(self, Q, cache_layer, slot, pos, out, sink, H, G, dim, vdim, scale, chunk=0, window=0,
                        n_split=None, bias_exp: float = 0.0, unit_sink: bool = False):
         """n_split None: enough blocks per (token, kv head) to fill the GPU when the step has few tokens, 1 for prompts;
@@ -453,16 +489,28 @@ class LayerOps:
         decay_logits (T, H dim) with bonus (H, dim): a decay per key channel w = exp(-exp(decay_logits)) and
         out = S^T q + (sum_i q_i bonus_i k_i) v with S the state before the token, then S <- diag(w) S + k v^T;
         part_len > 0 (with decay_logits, a prompt step): sequences longer than that are walked in parts of part_len
-        tokens at the same time (the state is linear in its start state, so the parts' contributions chain exactly)"""
+        tokens at the same time (the state is linear in its start state, so the parts' contributions chain exactly);
+        decay_logits with delta (and no bonus): the delta rule with a decay per key channel of every head,
+        w = exp(-exp(A_log) softplus(decay_logits + dt_bias)), S <- diag(w) S before the write and the read-out; a prompt
+        step walks 8 tokens at a time"""
         _, seqs, G = ctx.seq_tables()
         T, Hk = q.shape[0], H // rep
         # a prompt step does the per-token work (activation, unit lengths, k . q, decay, beta) in one parallel pass first
-        if decay_logits is not None:
+        max_rows = 1
+        if decay_logits is not None and delta:
+            prep = None
+            if T > SKINNY_ROWS:
+                lanes = 1
+                while lanes * 8 < dim:
+                    lanes *= 2
+                max_rows = max(n for _, n, _, _ in ctx.segments) if ctx.segments else 1
+                prep = self.empty(((T // 8 + G + 1) * H * (25 * 8 * lanes + 128),))
+        elif decay_logits is not None:
             prep = self.empty((T * (3 * H * dim + H),)) if T > SKINNY_ROWS else None
         else:
             prep = self.empty((T * (2 * Hk * dim + Hk + 2 * H),)) if T > SKINNY_ROWS else None
         scratch, n_parts = None, 0
-        if decay_logits is not None and prep is not None and part_len > 0 and ctx.segments:
+        if decay_logits is not None and not delta and prep is not None and part_len > 0 and ctx.segments:
             n_parts = max(-(-n // part_len) for _, n, _, _ in ctx.segments)
             if n_parts > 1:
                 lanes = 1
@@ -475,7 +523,7 @@ class LayerOps:
             vdim, int(act), float(unit_eps), float(q_scale), N.ptr(decay_const), N.ptr(a), a.stride(0) if a is not None else 0,
             N.ptr(A_log), N.ptr(dt_bias), N.ptr(b), b.stride(0) if b is not None else 0, int(delta), int(dt_in), N.ptr(skip),
             N.ptr(decay_logits), decay_logits.stride(0) if decay_logits is not None else 0, N.ptr(bonus),
-            N.ptr(prep), int(part_len) if scratch is not None else 0, n_parts, N.ptr(scratch), T, self.s),
+            N.ptr(prep), int(part_len) if scratch is not None else 0, n_parts, N.ptr(scratch), max_rows, T, self.s),
             "lm_linear_state")
 
     def head_post(self, o, out, *, dv, gate=None, gate_per_head=False, gate_silu=False, w=None, eps=0.0, span=0,
@@ -486,25 +534,26 @@ class LayerOps:
                                             int(gate_per_head), int(gate_silu), dv, n, float(scale), out.data_ptr(),
                                             out.stride(0), int(gate_first), T, self.s), "lm_head_post")
 
-    def glu_clamp(self, G, U, limit, alpha, Y, up_offset: float = 1.0, cubic: float = 0.0):
+    def glu_clamp(self, G, U, limit, alpha, Y, up_offset: float = 1.0, cubic: float = 0.0, relu: bool = False):
         """Y = g sigmoid(alpha (g + cubic g^3)) (u + up_offset), g = min(G, limit), u = clamp(U, +-limit); limit inf,
-        alpha 1 and up_offset 0 give the plain silu-gated unit; GELU_TANH_ALPHA and GELU_TANH_CUBIC the tanh form of gelu"""
+        alpha 1 and up_offset 0 give the plain silu-gated unit; GELU_TANH_ALPHA and GELU_TANH_CUBIC the tanh form of gelu;
+        relu: max(g, 0) (u + up_offset)"""
         T, n = G.shape
         self._ok(self.lib.b200_lm_glu_clamp(G.data_ptr(), G.stride(0), U.data_ptr(), U.stride(0), float(limit),
-                                            float(alpha), float(cubic), float(up_offset), Y.data_ptr(), Y.stride(0), n, T,
-                                            self.s),
+                                            float(alpha), float(cubic), float(up_offset), int(relu), Y.data_ptr(), Y.stride(0),
+                                            n, T, self.s),
                  "lm_glu_clamp")
 
     def glu_clamp_bf16(self, G, U, limit, alpha, up_offset: float = 1.0, live: Optional[torch.Tensor] = None,
-                       cubic: float = 0.0) -> torch.Tensor:
+                       cubic: float = 0.0, relu: bool = False) -> torch.Tensor:
         """the gated activation written as bf16 operand rows (T, ceil64(n)) of the next tensor-core product; live (T,)
         int32: rows with a negative entry (padding of sorted expert segments) become zeros without being read"""
         T, n = G.shape
         Kp = (n + 63) // 64 * 64
         Y = self.empty((T, Kp), torch.bfloat16)
         self._ok(self.lib.b200_lm_glu_clamp_bf16(G.data_ptr(), G.stride(0), U.data_ptr(), U.stride(0), float(limit),
-                                                 float(alpha), float(cubic), float(up_offset), Y.data_ptr(), n, Kp,
-                                                 N.ptr(live), T, self.s),
+                                                 float(alpha), float(cubic), float(up_offset), int(relu), Y.data_ptr(), n,
+                                                 Kp, N.ptr(live), T, self.s),
                  "lm_glu_clamp_bf16")
         return Y
 
