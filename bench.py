@@ -511,7 +511,7 @@ def c4_leg(dev, args):
 
 
 # ------------------------------------------------------------------------------------------------------------
-# `--design buzopel | sonulorn | lilosun | vadelix`: prefill and decode throughput of a decoder design assembled from decoder_blocks
+# `--design buzopel | sonulorn | lilosun | vadelix | futidra`: prefill and decode throughput of a decoder design assembled from decoder_blocks
 # over the layer ops (Buzopel: latent attention + expert mixture; Sonulorn: sink attention, matrix-state mixers and a
 # clamped gated feed-forward behind one shared input projection; Lilosun: windowed gated latent attention and state-space
 # mixers in scaled pre-norm layers with a grouped expert mixture — also beside Buzopel, the closest design on the same
@@ -705,11 +705,60 @@ def _vadelix_account(m, z, T):
     return act_w, other, mix_flops
 
 
+# Futidra at the layer sizes of the designs above: windowed latent attention (one layer borrows the latent of the other),
+# a delta rule with a decay per key channel, windowed grouped attention whose values are the keys, relu-gated units.  Beside
+# it Sonulorn at equal width, depth, head sizes, feed-forward and window: the closest design on the same engine (grouped
+# attention over a bounded range of keys, a gated delta rule behind short convolutions, gated dense units).
+FUTIDRA_SIZES = {
+    "2048w": dict(SONULORN_SIZES["2048w"], kv_rank=512, q_rank=1536, window=1024, rank=128),
+    "4096w": dict(SONULORN_SIZES["4096w"], kv_rank=512, q_rank=1536, window=1024, rank=128),
+}
+
+
+def _futidra_config(z):
+    H, d = z["heads"], z["dim"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    lat = {"heads": H, "dim": d, "vdim": d, "kv_rank": z["kv_rank"], "q_rank": z["q_rank"], "mask": {"size": z["window"]},
+           "scale": d ** -0.5}
+    delta = {"heads": H, "kv_heads": max(1, H // 2), "dim": d, "vdim": d, "conv": 4, "a_rank": z["rank"], "g_rank": z["rank"]}
+    att = {"heads": H, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "mask": {"size": z["window"]}, "scale": d ** -0.5,
+           "rot": {"base": 500000.0, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    layers = [{"type": "latent_attention", "mixer": lat, "mlp": mlp}, {"type": "channel_delta", "mixer": delta, "mlp": mlp},
+              {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": mlp},
+              {"type": "attention", "mixer": att, "mlp": mlp}]
+    return {"architecture": "Futidra", "vocab": z["vocab"], "width": z["width"], "layers": layers[:z["layers"]],
+            "norm": {"eps": 1e-5}, "postln_alpha": 1.7}
+
+
+def _futidra_model(z, dev):
+    from mlx_vlm_b200.models.futidra import Model as FModel, ModelConfig as FConfig
+    return FModel(FConfig.from_dict(_futidra_config(z)), device=dev).init_random(0)
+
+
+def _futidra_account(m, z, T):
+    from mlx_vlm_b200.models.decoder_blocks import GroupedAttention, LatentAttention
+    W = z["width"]
+    act_w, other, mix_flops = 0, 8 * m.state_floats, 0.0      # the fp32 state is read and written once per token
+    for L in m.layers:
+        x = L.mixer
+        act_w += sum(t.numel() for t in x.w.values()) + (3 * L.ff.ff * W if L.ff is not None else 0)
+        if isinstance(x, (GroupedAttention, LatentAttention)):
+            # visible keys of a query, averaged over the prompt; a decoded token after it reads a whole window
+            mean_seen = sum(min(p + 1, x.window or p + 1) for p in range(T)) / T
+            per_key = x.row_dim + x.kv_rank if isinstance(x, LatentAttention) else x.dim + x.vdim
+            mix_flops += 2 * x.H * per_key * mean_seen
+            other += 2 * x.kv_dim * min(x.window or T, T)
+        else:
+            mix_flops += 6 * x.H * x.dim * x.vdim
+    return act_w, other, mix_flops
+
+
 # design -> (sizes, model factory, byte / flop accounting, closest design on the same engine measured beside it or None)
 DESIGNS = {"buzopel": (DESIGN_SIZES, _buzopel_model, _buzopel_account, None),
            "sonulorn": (SONULORN_SIZES, _sonulorn_model, _sonulorn_account, None),
            "lilosun": (LILOSUN_SIZES, _lilosun_model, _lilosun_account, ("buzopel_equal_size", _buzopel_model, _buzopel_account)),
-           "vadelix": (VADELIX_SIZES, _vadelix_model, _vadelix_account, ("lilosun_equal_size", _lilosun_model, _lilosun_account))}
+           "vadelix": (VADELIX_SIZES, _vadelix_model, _vadelix_account, ("lilosun_equal_size", _lilosun_model, _lilosun_account)),
+           "futidra": (FUTIDRA_SIZES, _futidra_model, _futidra_account, ("sonulorn_equal_size", _sonulorn_model, _sonulorn_account))}
 
 
 def _measure_layered(m, account, z, T, n_dec, rows, ids, args, timed, hbm, tpk):
@@ -840,7 +889,7 @@ def main():
     ap.add_argument("--no-mega", action="store_true")
     ap.add_argument("--mega-mode", type=int, default=None,
                     help="decode kernel: 0 per-phase kernels, 1 k_mega (CUDA cores), 2 k_mega_tc (tcgen05)")
-    ap.add_argument("--design", default=None, choices=["buzopel", "sonulorn", "lilosun", "vadelix"],
+    ap.add_argument("--design", default=None, choices=["buzopel", "sonulorn", "lilosun", "vadelix", "futidra"],
                     help="instead of the default workload: prefill / decode throughput of this decoder design at "
                          "layer sizes of real models, beside the closest existing model at equal size")
     ap.add_argument("--design-sizes", default="", help="comma-separated subset of the sizes (default: all)")

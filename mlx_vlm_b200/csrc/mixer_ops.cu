@@ -984,7 +984,7 @@ __global__ void state_parts_chain_kernel(StateP p, int P) {
 // and head), delta_chunk_kernel walks the chunks.  The chain from chunk to chunk then holds ONE reduction over the lanes of
 // a column for DC_C tokens, and the 2 DC_C sums of a column are reduced together (each lane ends with its own sums).
 // All arithmetic is fp32.  A chunk past the end of its sequence is filled with tokens that change nothing (g = 1, k = q = 0).
-constexpr int DC_C = 8;
+constexpr int DC_C = 8, DC_THREADS = 128;
 struct DeltaChunkP {
   const float* q; long ldq;         // activated
   const float* k; long ldk;
@@ -1002,94 +1002,6 @@ struct DeltaChunkP {
 };
 // the first chunk of sequence g of the step: no two sequences share one (a sequence has at most rows / C + 1 of them)
 __device__ __forceinline__ long first_chunk(const int* seqs, int g) { return seqs[2 * g] / DC_C + g; }
-template <int P>
-__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(DeltaChunkP p) {
-  constexpr int C = DC_C, D = P * LS_R, NCH = (D + 31) / 32, TILE = (3 * C + 1) * D + 2 * C * C;
-  __shared__ float sA[4][C * C], sB[4][C * C], sT[4][C * C];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, seq = blockIdx.z;
-  const int h = blockIdx.y * 4 + warp, hk = h / p.rep;
-  const int start = p.seqs[2 * seq] + blockIdx.x * C, nc = min(C, p.seqs[2 * seq + 1] - (int)blockIdx.x * C);
-  if (nc <= 0 || h >= p.H) return;             // whole warps
-  float* tile = p.tiles + ((first_chunk(p.seqs, seq) + blockIdx.x) * p.H + h) * TILE;
-  float ik[C], iq[C];
-#pragma unroll
-  for (int t = 0; t < C; ++t) {
-    float sk = 0.f, sq = 0.f;
-    if (t < nc) {
-      const float* kr = p.k + (long)(start + t) * p.ldk + (long)hk * p.dim;
-      const float* qr = p.q + (long)(start + t) * p.ldq + (long)hk * p.dim;
-      for (int i = lane; i < p.dim; i += 32) { sk = fmaf(kr[i], kr[i], sk); sq = fmaf(qr[i], qr[i], sq); }
-    }
-    ik[t] = 1.0f / sqrtf(warp_sum(sk) + p.unit_eps);
-    iq[t] = p.q_scale / sqrtf(warp_sum(sq) + p.unit_eps);
-  }
-  const float A = expf(bf2f(p.A_log[h]));
-  float acc[C * C];                            // entry (t, s): A_ts below the diagonal; B_ts is kept in bcc
-  float bcc[C * C];
-#pragma unroll
-  for (int e = 0; e < C * C; ++e) acc[e] = bcc[e] = 0.f;
-#pragma unroll 1
-  for (int n = 0; n < NCH; ++n) {
-    const int i = n * 32 + lane;
-    float k[C], q[C], g[C];
-#pragma unroll
-    for (int t = 0; t < C; ++t) {
-      const bool ok = t < nc && i < p.dim;
-      k[t] = ok ? p.k[(long)(start + t) * p.ldk + (long)hk * p.dim + i] * ik[t] : 0.f;
-      q[t] = ok ? p.q[(long)(start + t) * p.ldq + (long)hk * p.dim + i] * iq[t] : 0.f;
-      g[t] = 1.f;
-      if (ok) g[t] = expf(-A * softplus_exact(p.x[(long)(start + t) * p.ldx + (long)h * p.dim + i] + bf2f(p.dt_bias[(long)h * p.dim + i])));
-    }
-#pragma unroll
-    for (int s = 0; s < C; ++s) {
-      float kd = k[s];
-      bcc[s * C + s] = fmaf(q[s], kd, bcc[s * C + s]);
-#pragma unroll
-      for (int t = s + 1; t < C; ++t) {
-        kd *= g[t];
-        acc[t * C + s] = fmaf(k[t], kd, acc[t * C + s]);
-        bcc[t * C + s] = fmaf(q[t], kd, bcc[t * C + s]);
-      }
-      if (i < D) tile[(2 * C + s) * D + i] = kd;
-    }
-    float G = 1.f;
-#pragma unroll
-    for (int t = 0; t < C; ++t) {
-      G *= g[t];
-      if (i < D) { tile[t * D + i] = G * k[t]; tile[(C + t) * D + i] = G * q[t]; }
-    }
-    if (i < D) tile[3 * C * D + i] = G;
-  }
-#pragma unroll
-  for (int t = 0; t < C; ++t)
-#pragma unroll
-    for (int s = 0; s <= t; ++s) {
-      const float a = s < t ? warp_sum(acc[t * C + s]) : 0.f, b = warp_sum(bcc[t * C + s]);
-      if (lane == 0) { sA[warp][t * C + s] = a; sB[warp][t * C + s] = b; }
-    }
-  __syncwarp();
-  if (lane < C) {                              // lane j: column j of T by forward substitution, then of B T
-    float col[C];
-#pragma unroll
-    for (int t = 0; t < C; ++t) {
-      const float beta = t < nc ? sigmoid_exact(p.b[(long)(start + t) * p.ldb + h]) : 0.f;
-      float v = t == lane ? 1.f : 0.f;
-#pragma unroll
-      for (int s = 0; s < t; ++s) v = fmaf(-sA[warp][t * C + s], col[s], v);
-      col[t] = beta * v;
-      sT[warp][t * C + lane] = col[t];
-    }
-    float* M = tile + (3 * C + 1) * D;
-#pragma unroll
-    for (int t = 0; t < C; ++t) {
-      float m = 0.f;
-#pragma unroll
-      for (int s = 0; s <= t; ++s) m = fmaf(sB[warp][t * C + s], col[s], m);
-      M[t * C + lane] = col[t];
-      M[C * C + t * C + lane] = m;
-    }
-  }
-}
 // N sums held by every one of 2 O lanes: halve the sums a lane holds and the lanes that share them, step by step; once a
 // lane holds one, the last steps add.  Lane r of the group ends with the sums r N / (2 O) .. of the N
 template <int N, int O>
@@ -1109,16 +1021,113 @@ __device__ __forceinline__ void reduce_scatter(float* a, int lane) {
     }
   }
 }
+// a row of D = 8 P numbers in a tile: lane r of a column owns numbers 8 r .. 8 r + 7, stored as two vectors of four, all lanes'
+// first vectors and then all lanes' second ones, so that a warp's 16-byte loads are contiguous.  The number at a position:
+template <int P>
+__device__ __forceinline__ int tile_number(int at) { return (at >> 2) % P * LS_R + (at >> 2) / P * 4 + (at & 3); }
+template <int P>
+__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(DeltaChunkP p) {
+  constexpr int C = DC_C, D = P * LS_R, NCH = (D + 31) / 32, TILE = (3 * C + 1) * D + 2 * C * C;
+  constexpr int NA = C * (C - 1) / 2;          // sums: A_ts at t (t - 1) / 2 + s, then B_ts at NA + t (t + 1) / 2 + s
+  static_assert(NA + C * (C + 1) / 2 == C * C, "");
+  __shared__ float sums[4][C * C], inv[4][2 * C];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, seq = blockIdx.z;
+  const int h = blockIdx.y * 4 + warp, hk = h / p.rep;
+  const int start = p.seqs[2 * seq] + blockIdx.x * C, nc = min(C, p.seqs[2 * seq + 1] - (int)blockIdx.x * C);
+  if (nc <= 0 || h >= p.H) return;             // whole warps
+  float* tile = p.tiles + ((first_chunk(p.seqs, seq) + blockIdx.x) * p.H + h) * TILE;
+  const float* kp = p.k + (long)start * p.ldk + (long)hk * p.dim;
+  const float* qp = p.q + (long)start * p.ldq + (long)hk * p.dim;
+  {
+    float ss[2 * C];
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      ss[t] = ss[C + t] = 0.f;
+      if (t < nc)
+        for (int i = lane; i < p.dim; i += 32) {
+          const float a = kp[(long)t * p.ldk + i], b = qp[(long)t * p.ldq + i];
+          ss[t] = fmaf(a, a, ss[t]); ss[C + t] = fmaf(b, b, ss[C + t]);
+        }
+    }
+    reduce_scatter<2 * C, 16>(ss, lane);       // lane l ends with sum l / 2
+    if ((lane & 1) == 0) inv[warp][lane >> 1] = (lane >> 1 < C ? 1.0f : p.q_scale) / sqrtf(ss[0] + p.unit_eps);
+  }
+  __syncwarp();
+  const float A = expf(bf2f(p.A_log[h]));
+  float acc[C * C];
+#pragma unroll
+  for (int e = 0; e < C * C; ++e) acc[e] = 0.f;
+#pragma unroll 1
+  for (int n = 0; n < NCH; ++n) {
+    const int at = n * 32 + lane, i = at < D ? tile_number<P>(at) : D;
+    float k[C], q[C], g[C];
+    const float dtb = i < p.dim ? bf2f(p.dt_bias[(long)h * p.dim + i]) : 0.f;
+    const float* xp = p.x + (long)start * p.ldx + (long)h * p.dim + i;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      const bool ok = t < nc && i < p.dim;
+      k[t] = ok ? kp[(long)t * p.ldk + i] * inv[warp][t] : 0.f;
+      q[t] = ok ? qp[(long)t * p.ldq + i] * inv[warp][C + t] : 0.f;
+      g[t] = ok ? xp[(long)t * p.ldx] : 0.f;
+    }
+#pragma unroll
+    for (int t = 0; t < C; ++t) g[t] = (t < nc && i < p.dim) ? expf(-A * softplus_exact(g[t] + dtb)) : 1.f;
+#pragma unroll
+    for (int s = 0; s < C; ++s) {
+      float kd = k[s];
+      acc[NA + s * (s + 1) / 2 + s] = fmaf(q[s], kd, acc[NA + s * (s + 1) / 2 + s]);
+#pragma unroll
+      for (int t = s + 1; t < C; ++t) {
+        kd *= g[t];
+        acc[t * (t - 1) / 2 + s] = fmaf(k[t], kd, acc[t * (t - 1) / 2 + s]);
+        acc[NA + t * (t + 1) / 2 + s] = fmaf(q[t], kd, acc[NA + t * (t + 1) / 2 + s]);
+      }
+      if (at < D) tile[(2 * C + s) * D + at] = kd;
+    }
+    float G = 1.f;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      G *= g[t];
+      if (at < D) { tile[t * D + at] = G * k[t]; tile[(C + t) * D + at] = G * q[t]; }
+    }
+    if (at < D) tile[3 * C * D + at] = G;
+  }
+  reduce_scatter<C * C, 16>(acc, lane);        // lane l ends with sums 2 l, 2 l + 1
+  sums[warp][2 * lane] = acc[0];
+  sums[warp][2 * lane + 1] = acc[1];
+  __syncwarp();
+  if (lane < C) {                              // lane j: column j of T by forward substitution, then of B T
+    float col[C];
+    float* M = tile + (3 * C + 1) * D;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      const float beta = t < nc ? sigmoid_exact(p.b[(long)(start + t) * p.ldb + h]) : 0.f;
+      float v = t == lane ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) v = fmaf(-sums[warp][t * (t - 1) / 2 + s], col[s], v);
+      col[t] = beta * v;
+      M[t * C + lane] = col[t];
+    }
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      float m = 0.f;
+#pragma unroll
+      for (int s = 0; s <= t; ++s) m = fmaf(sums[warp][NA + t * (t + 1) / 2 + s], col[s], m);
+      M[C * C + t * C + lane] = m;
+    }
+  }
+}
 template <int P, int NC>
-__global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) {
-  // a column belongs to P lanes of one warp, NC neighbouring columns to the same lanes; a warp holds CW columns.  Chunk
-  // tiles are copied ahead (cp.async, two buffers); the rows of k~, q~, k^ are laid out LS_RS apart per lane (no bank conflicts)
-  constexpr int C = DC_C, D = P * LS_R, TILE = (3 * C + 1) * D + 2 * C * C, LD = P * LS_RS, ROWS = 3 * C + 1;
-  constexpr int NW = LS_THREADS / 32, CW = 32 / P * NC, PAIRS = (C * CW + 31) / 32, BUF = ROWS * LD + 2 * C * C;
+__global__ void __launch_bounds__(DC_THREADS) delta_chunk_kernel(DeltaChunkP p) {
+  // a column belongs to P lanes of one warp, NC neighbouring columns to the same lanes (the rows of k~, q~, k^ that a lane
+  // loads from shared memory, which is what bounds the walk, serve all of them); a warp holds CW columns.  Chunk tiles are
+  // copied ahead (cp.async, two buffers)
+  constexpr int C = DC_C, D = P * LS_R, TILE = (3 * C + 1) * D + 2 * C * C, ROWS = 3 * C + 1;
+  constexpr int NW = DC_THREADS / 32, CW = 32 / P * NC, PAIRS = (C * CW + 31) / 32;
   constexpr int NV = 2 * C;                    // sums per column, reduced over P lanes: a lane ends with NL of them
   constexpr int NL = P >= NV ? 1 : NV / P;
   extern __shared__ __align__(16) float sm[];
-  float* red = sm + 2 * BUF + (threadIdx.x >> 5) * (CW * (NV + 2 * C));       // this warp's: sums [CW][2C], w [CW][C], u [CW][C]
+  float* red = sm + 2 * TILE + (threadIdx.x >> 5) * (CW * (NV + 2 * C));       // this warp's: sums [CW][2C], w [CW][C], u [CW][C]
   float* wv = red + CW * NV;
   float* us = wv + CW * C;
   const int seq = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1136,13 +1145,10 @@ __global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) 
   const float* tiles = p.tiles + (first_chunk(p.seqs, seq) * p.H + h) * TILE;
   auto fetch = [&](int c) {
     const float* t = tiles + (long)c * p.H * TILE;
-    float* d = sm + (c & 1) * BUF;
-    for (int e = threadIdx.x; e < TILE / 4; e += LS_THREADS) {
-      const int f = e * 4, row = f / D, i = f % D;
-      float* to = row < ROWS ? d + row * LD + (i / LS_R) * LS_RS + i % LS_R : d + ROWS * LD + (f - ROWS * D);
-      const unsigned a = (unsigned)__cvta_generic_to_shared(to);
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(t + f) : "memory");
-    }
+    const unsigned d = (unsigned)__cvta_generic_to_shared(sm + (c & 1) * TILE);
+#pragma unroll 4
+    for (int f = threadIdx.x * 4; f < TILE; f += DC_THREADS * 4)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d + f * 4), "l"(t + f) : "memory");
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   float vn[PAIRS];                             // the values of the lane's (token, column) pairs, one chunk ahead
@@ -1159,12 +1165,12 @@ __global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) 
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                           // this chunk's tile is here, and everyone has left the other buffer
     if (c + 1 < n_chunks) fetch(c + 1);
-    const float* B = sm + (c & 1) * BUF;
+    const float* B = sm + (c & 1) * TILE;
     float a[NC][NV];
 #pragma unroll
     for (int t = 0; t < NV; ++t) {             // rows 0 .. C-1: k~, C .. 2C-1: q~
-      const float* x = B + t * LD + r * LS_RS;
-      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float* x = B + t * D + r * 4;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4 * P);
       const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
       for (int j = 0; j < NC; ++j) {
@@ -1188,7 +1194,7 @@ __global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) 
       if (e < C * CW) wv[cc * C + t] = vn[n] - red[cc * NV + t];
     }
     __syncwarp();
-    const float* TT = B + ROWS * LD;
+    const float* TT = B + ROWS * D;
 #pragma unroll
     for (int n = 0; n < PAIRS; ++n) {          // u_t = T_t . w,  o_t = S^T q~_t + (B T)_t . w
       const int e = lane + 32 * n, t = e / CW, cc = e % CW;
@@ -1208,8 +1214,8 @@ __global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) 
     if (c + 1 < n_chunks) request_v(c + 1);
     __syncwarp();
     {
-      const float* x = B + 3 * C * LD + r * LS_RS;
-      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float* x = B + 3 * C * D + r * 4;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4 * P);
       const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
       for (int j = 0; j < NC; ++j)
@@ -1218,8 +1224,8 @@ __global__ void __launch_bounds__(LS_THREADS) delta_chunk_kernel(DeltaChunkP p) 
     }
 #pragma unroll
     for (int t = 0; t < C; ++t) {
-      const float* x = B + (2 * C + t) * LD + r * LS_RS;
-      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+      const float* x = B + (2 * C + t) * D + r * 4;
+      const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4 * P);
       const float x_[LS_R] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
       for (int j = 0; j < NC; ++j) {
@@ -1404,22 +1410,24 @@ __global__ void sink_softmax_bf16_kernel(const float* __restrict__ S, long lds, 
 
 unsigned long long g_sink_attr_f32 = 0, g_sink_attr_bf16 = 0;
 
-// all chunks' tiles, then the walk.  Two columns per lane set when that still gives every SM a block.
+// all chunks' tiles, then the walk: as many columns per lane as still leave the GPU enough blocks
 template <int P>
 int delta_chunks(const DeltaChunkP& p, int n_seq, int max_rows, cudaStream_t cs) {
   static unsigned long long attr = 0;
-  constexpr int BUF = (3 * DC_C + 1) * P * LS_RS + 2 * DC_C * DC_C;
-  auto smem = [](int nc) { return (size_t)(2 * BUF + LS_THREADS / 32 * (32 / P * nc) * 4 * DC_C) * sizeof(float); };
+  constexpr int TILE = (3 * DC_C + 1) * P * LS_R + 2 * DC_C * DC_C, cols = DC_THREADS / P;
+  auto smem = [](int nc) { return (size_t)(2 * TILE + cols * nc * 4 * DC_C) * sizeof(float); };
   if (first_use_on_device(&attr)) {
     B200_CUDA(cudaFuncSetAttribute(delta_chunk_kernel<P, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem(1)));
     B200_CUDA(cudaFuncSetAttribute(delta_chunk_kernel<P, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem(2)));
+    B200_CUDA(cudaFuncSetAttribute(delta_chunk_kernel<P, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem(4)));
   }
   delta_chunk_prep_kernel<P><<<dim3(cdiv(max_rows, DC_C), cdiv(p.H, 4), n_seq), 128, 0, cs>>>(p);
   B200_CHECK_LAUNCH();
-  const int cols = LS_THREADS / P;
-  const long two = (long)n_seq * p.H * cdiv(p.vdim, 2 * cols);
-  if (two >= 148) delta_chunk_kernel<P, 2><<<dim3(n_seq, p.H, cdiv(p.vdim, 2 * cols)), LS_THREADS, smem(2), cs>>>(p);
-  else delta_chunk_kernel<P, 1><<<dim3(n_seq, p.H, cdiv(p.vdim, cols)), LS_THREADS, smem(1), cs>>>(p);
+  auto grid = [&](int nc) { return dim3(n_seq, p.H, cdiv(p.vdim, nc * cols)); };
+  auto blocks = [&](int nc) { return (long)n_seq * p.H * cdiv(p.vdim, nc * cols); };
+  if (blocks(4) >= 2 * 148) delta_chunk_kernel<P, 4><<<grid(4), DC_THREADS, smem(4), cs>>>(p);
+  else if (blocks(2) >= 96) delta_chunk_kernel<P, 2><<<grid(2), DC_THREADS, smem(2), cs>>>(p);
+  else delta_chunk_kernel<P, 1><<<grid(1), DC_THREADS, smem(1), cs>>>(p);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }
