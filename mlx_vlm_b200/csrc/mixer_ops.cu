@@ -1425,7 +1425,7 @@ int delta_chunks(const DeltaChunkP& p, int n_seq, int max_rows, cudaStream_t cs)
   B200_CHECK_LAUNCH();
   auto grid = [&](int nc) { return dim3(n_seq, p.H, cdiv(p.vdim, nc * cols)); };
   auto blocks = [&](int nc) { return (long)n_seq * p.H * cdiv(p.vdim, nc * cols); };
-  if (blocks(4) >= 2 * 148) delta_chunk_kernel<P, 4><<<grid(4), DC_THREADS, smem(4), cs>>>(p);
+  if (blocks(4) >= 120) delta_chunk_kernel<P, 4><<<grid(4), DC_THREADS, smem(4), cs>>>(p);
   else if (blocks(2) >= 96) delta_chunk_kernel<P, 2><<<grid(2), DC_THREADS, smem(2), cs>>>(p);
   else delta_chunk_kernel<P, 1><<<grid(1), DC_THREADS, smem(1), cs>>>(p);
   B200_CHECK_LAUNCH();

@@ -605,6 +605,10 @@ OTHER = {
     "equal ranks and sizes, wide heads, an odd vocabulary": config(
         [layer("channel_delta", delta(heads=2, kv_heads=1, dim=72, vdim=72, conv=4, a_rank=16, g_rank=16)),
          layer("attention", att(heads=3, kv_heads=1, dim=72, dims=40, window=64))], width=72, vocab=257),
+    "nothing cached": config([layer("channel_delta", delta(heads=3, kv_heads=1, dim=11, vdim=13, conv=6), 25),
+                              layer("channel_delta", delta(heads=2, kv_heads=2, dim=33, vdim=10, conv=2), None)], width=52, vocab=77),
+    "no state": config([layer("attention", att(heads=5, kv_heads=5, dim=18, dims=6, window=23), 28),
+                        layer("latent_attention", lat(heads=6, dim=14, vdim=18, kv_rank=36, window=29), None)], width=60, vocab=89),
     "many heads, odd sizes": config(
         [layer("channel_delta", delta(heads=12, kv_heads=4, dim=5, vdim=7, a_rank=3, g_rank=5)),
          layer("latent_attention", lat(heads=11, dim=5, vdim=3, kv_rank=17, q_rank=9, window=8), 33)], width=45, vocab=61),
