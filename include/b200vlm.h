@@ -326,9 +326,10 @@ int b200_gemm_wt_f32(const void* X, long ldx, const void* W, long ldw, const voi
 int b200_gemm_wt_f32_grouped(const void* X, long ldx, const void* W, long ldw, float* C32, long ldc32,
                              const int* tile_group, int n_tiles, int n_groups, int N, int K_w, void* stream);
 /* the per-head projections of one token set in ONE launch: head g multiplies columns [g * x_group_cols, + K_w) of
- * X [T, x_cols] (bf16; K_w % 64 == 0) by W[g] [N, K_w] and writes columns [g * c_group_cols, + N) of C32 */
+ * X [T, x_cols] (bf16; K_w % 64 == 0) by W[g] [N, K_w] and writes columns [g * c_group_cols, + N) of C32; n_parts = 2: the
+ * columns of a head are the [hi | lo] halves of K_w fp32 numbers, both multiplied by W[g] */
 int b200_gemm_wt_f32_heads(const void* X, long ldx, int x_cols, int x_group_cols, const void* W, long ldw, float* C32,
-                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, void* stream);
+                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, int n_parts, void* stream);
 
 /* ------------------------------------------------------------------------- */
 /* Lock-step batched decode (continuous batching; generate/ar.py:929-1390        */
@@ -377,6 +378,23 @@ float b200_engine_last_decode_ms(const b200_engine* e);
 /* ------------------------------------------------------------------------- */
 /* x[t] = embed[tokens[t]] * scale */
 int b200_lm_embed(const int* tokens, const void* embed, float scale, float* x, int T, int W, int vocab, void* stream);
+/* x[t] = embed[tokens[t]] * scale + bigram[(prev mul_prev + cur mul_cur) mod buckets] (row `buckets` at position 0); the token
+ * before a step's first one is kept in the first number of the slot's state (its bits), which the step advances (single: every
+ * sequence of the step is one token, in the same launch).  keep (may be NULL): a second copy of x; norm_w (may be NULL):
+ * xn = x / sqrt(mean(x^2) + eps) * norm_w, xb (may be NULL): xn as bf16 rows of ldb >= W columns, zero-padded */
+int b200_lm_embed_bigram(const int* tokens, const void* embed, float scale, const void* bigram, int buckets, long mul_prev,
+                         long mul_cur, float* state, long slot_stride, const int* slot, const int* pos, const int* first,
+                         const int* seqs, int n_seq, int single, float* x, float* keep, const void* norm_w, float eps, float* xn,
+                         void* xb, long ldb, int T, int W, int vocab, void* stream);
+/* x[t] += sum over nb <= 3 branches of m_b N_b(y_b[t]) (+ extra[t]), N_b(y) = y / sqrt(mean(y^2) + eps) * w_b, or y itself where
+ * w_b is NULL; then out[t] = x / sqrt(mean(x^2) + eps) * norm_w (norm_w NULL: no norm).  xb (may be NULL): bf16 rows of
+ * ldb >= N columns, zero-padded, of out or, without norm_w, of x */
+int b200_lm_close_rows(float* x, long ldx, int nb, const float* y0, long ldy0, const void* w0, float m0, const float* y1, long ldy1,
+                       const void* w1, float m1, const float* y2, long ldy2, const void* w2, float m2, const float* extra,
+                       long lde, const void* norm_w, float eps, float* out, long ldo, void* xb, long ldb, int T, int N, void* stream);
+/* out[t][i] = gelu(z[t][i]) (tanh form) * table[tokens[t]][i], bf16 rows of ldo >= n columns, zero-padded */
+int b200_lm_table_gate_bf16(const float* z, long ldz, const void* table, long ld_table, int table_rows, const int* tokens, void* out,
+                            int n, int ldo, int T, void* stream);
 /* cs[t][i] = amp * (cos, sin)(pos[t] * inv_freq[i]), angle in double precision; inv_freq[half] doubles on the device */
 int b200_lm_rope_table(const int* pos, const double* inv_freq, float* cs, int T, int half, float amp, void* stream);
 /* n = y / sqrt(mean(y^2) + eps) * (w_offset + w); x = n or (add) x += n.  wgt != NULL: y row t is the weighted
@@ -429,10 +447,12 @@ int b200_lm_moe_group(const int* idx, int n_entries, int E, int* list, long list
  * list[b][0..count[b]), x row = entry / x_div, y row = entry.  epi 0 none, 1 relu^2, 2 p*tanh(v/p), 4 v*p.
  * skinny != 0: the decode kernels (weight rows streamed once for the few rows of X).  compact > 0 (skinny, with
  * counts): at most `compact` batches have rows, and only that many slices are launched (slice z = the z-th batch
- * whose count is not zero). */
+ * whose count is not zero).  One plain product (no batch, no lists) may have: X2, the rows multiplied are X + X2; epi 6,
+ * Y = gelu(product) (tanh form) * aux[aux_row[row]][n], aux a bf16 table of aux_rows rows. */
 int b200_lm_gemm_rows(const float* X, long ldx, long xb, const void* W, long ldw, long wb, const void* bias, float* Y,
                       long ldy, long yb, const int* list, long list_stride, const int* count, int x_div, int M, int N,
-                      int K, int batch, int epi, float epi_param, int round_x, int skinny, int compact, void* stream);
+                      int K, int batch, int epi, float epi_param, int round_x, int skinny, int compact, const float* X2, long ldx2,
+                      const void* aux, long ld_aux, const int* aux_row, int aux_rows, void* stream);
 /* operands of the tensor-core products of a prompt step (bf16 serving mode; the products are b200_gemm_wt_f32 with
  * one bf16 part): fp32 rows -> bf16 rows zero-padded to Kp columns (gather: src row = map[i] / div; relu2: the
  * experts' activation before the rounding); fp32 rows scattered to dst_map[i]; the causal softmax of score rows
@@ -487,19 +507,20 @@ int b200_lm_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* 
                      int qt_every, const void* vmix, const float* v_first, long ldvf, float* v_keep, long ldvk, int T,
                      void* stream);
 /* the same step with everything per head: qn_w / kn_w (bf16 [dim], or NULL): RMS norm (eps) of every query / key head times
- * ONE weight for all heads; then the rotation of pairs (i, i + rot_dims / 2) or (pairs) (2i, 2i + 1); V may be K's own rows */
+ * ONE weight for all heads (unit: such norms without a weight); then the rotation of pairs (i, i + rot_dims / 2) or (pairs) (2i, 2i + 1); V may be K's own rows */
 int b200_lm_head_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* V, long ldv, void* cache, int cache_bf16,
                           long slot_stride, long tok_stride, const int* slot, const int* pos, const float* cs, int H, int G,
-                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int T,
-                          void* stream);
+                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int unit,
+                          int T, void* stream);
 /* out[t][h] = softmax over the visible rows j of slot[t] (and the sink logit of head h, if any) of
  * scale * q[t][h] . K_j[h / (H/G)], times V_j; visible: max(block start of pos[t] (chunk > 0), pos[t] - window + 1
  * (window > 0), 0) <= j <= pos[t].  bias_exp > 0: 2^(-bias_exp (h + 1) / H) (pos[t] - j) is taken off the score;
- * unit_sink: the denominator also holds 1 (a sink logit of zero).  n_split > 1: key tiles dealt to n_split blocks, part [T][H][n_split][vdim + 2] */
+ * unit_sink: the denominator also holds 1 (a sink logit of zero); softcap > 0: a scaled score s becomes
+ * softcap tanh(s / softcap).  n_split > 1: key tiles dealt to n_split blocks, part [T][H][n_split][vdim + 2] */
 int b200_lm_sink_attention(const float* q, long ldq, const void* cache, int cache_bf16, long slot_stride, long tok_stride,
                            const int* slot, const int* pos, float* out, long ldo, const void* sink, int H, int G,
-                           int dim, int vdim, float scale, int chunk, int window, float bias_exp, int unit_sink, float* part,
-                           int n_split, int T, void* stream);
+                           int dim, int vdim, float scale, int chunk, int window, float bias_exp, int unit_sink, float softcap,
+                           float* part, int n_split, int T, void* stream);
 /* per head a (dim, vdim) state carried through each sequence: S <- decay S + k u^T, out = S^T q, u = v or
  * (delta) beta (v - (decay S)^T k); decay per head (decay_const) or exp(-exp(A_log) softplus(a + dt_bias)) per
  * token; beta = sigmoid(b) or 1; q, k shared by `rep` heads, optionally silu'd (act) and scaled to unit length.
@@ -524,11 +545,12 @@ int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, con
                          void* stream);
 /* operands of the tensor-core attention of a prompt step: out[(t, r)] = bf16 of q[t][r * dim .. + dim) padded to Kp;
  * P[(t, r)][j] = softmax over the visible keys key0 + j (and sink[r]) of scale * S[(t, r)][j], bf16, zero elsewhere;
- * split: P rows are [hi | lo] (Sp columns each), lo the rounding error of hi (the operand of a two-part product) */
+ * split: P rows are [hi | lo] (Sp columns each), lo the rounding error of hi (the operand of a two-part product);
+ * softcap > 0: scores become softcap tanh(scale S / softcap), which S then holds */
 int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int dim, void* out, int Kp, int T, void* stream);
-int b200_lm_sink_softmax_bf16(const float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
-                              int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, void* P,
-                              long ldp, int rows, int Sp, void* stream);
+int b200_lm_sink_softmax_bf16(float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
+                              int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, float softcap,
+                              void* P, long ldp, int rows, int Sp, void* stream);
 /* out[t][c] = scale * o[t][c] * [rsqrt(mean over c's group of `span` + eps)] * [w[c mod w_len]] * [act(gate)];
  * gate_first: the gate is applied before the norm (the mean square is that of the gated numbers) */
 int b200_lm_head_post(const float* o, long ldi, const float* gate, long ldg, const void* w, int w_len, float eps, int span,
@@ -543,6 +565,29 @@ int b200_lm_glu_clamp(const float* G, long ldg, const float* U, long ldu, float 
  * rows t with live[t] < 0 (the padding of sorted expert segments) are written as zeros and their inputs are not read */
 int b200_lm_glu_clamp_bf16(const float* G, long ldg, const float* U, long ldu, float limit, float alpha, float cubic, float up_off,
                            int relu, void* Y, int n, int Kp, const int* live, int T, void* stream);
+
+/* ------------------------------------------------------------------------- */
+/* Recurrent mixers (csrc/recurrent_ops.cu), same step layout                  */
+/* ------------------------------------------------------------------------- */
+/* gated linear recurrence per channel: log a = -c sigmoid(G_r + rb) softplus(lam); S <- a S + sqrt(1 - a^2) sigmoid(G_i + ib) u;
+ * out = S gelu(y) (tanh form).  G [T][n / bs][r: bs | i: bs] (scratch: overwritten with parts), state [n] per slot, zero at
+ * position 0.  out_bf16: bf16 rows of ldb >= n columns, zero-padded, instead of fp32 rows.  n_parts > 1: sequences are walked
+ * in parts of part_len rows at the same time; part: n_seq * n * (2 n_parts + 1) floats */
+int b200_lm_gated_recurrence(float* G, long ldg, int bs, const void* rb, const void* ib, const void* lam, float c, const float* u,
+                             long ldu, const float* y, long ldy, float* state, long slot_stride, const int* seqs, int n_seq,
+                             const int* slot, const int* pos, int n, float* out, long ldo, void* out_bf16, long ldb, int part_len,
+                             int n_parts, float* part, void* stream);
+/* matrix memory per head with exponential gates: i = cap tanh(gi / cap), f = logsigmoid(cap tanh(gf / cap)), m' = max(f + m, i),
+ * S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise, o = S^T (q_scale q) / (max(|n . q_scale q|, exp(-m')) + 1e-6), then
+ * o / sqrt(mean(o^2) + eps) per head * w * sigmoid(gate).  State per slot: [H][dim][vdim] | [H][dim] | [H].
+ * scratch (a prompt step; bytes as b200_lm_matrix_memory_scratch says): 64 tokens of a sequence at a time, all chunks at once;
+ * NULL: every sequence's rows are walked one after the other in one launch */
+long b200_lm_matrix_memory_scratch(int T, int n_seq, int H, int dim, int vdim);
+int b200_lm_matrix_memory(const float* q, long ldq, const float* k, long ldk, const float* v, long ldv, const float* gi, long ldi,
+                          const float* gf, long ldf, float cap, float q_scale, const float* gate, long ldg, const void* w, float eps,
+                          float* state, long slot_stride, const int* seqs, int n_seq, const int* slot, const int* pos, int H,
+                          int dim, int vdim, float* out, long ldo, void* out_bf16, long ldb, void* scratch, long scratch_bytes,
+                          int max_rows, int T, void* stream);
 
 #ifdef __cplusplus
 }

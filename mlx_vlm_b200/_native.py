@@ -112,6 +112,11 @@ LM_SIGNATURES = {
     "b200_abi_version": (_I, []),
     "b200_device_check": (_I, [_I, C.POINTER(_I)]),
     "b200_lm_embed": (_I, [_P, _P, _F, _P, _I, _I, _I, _P]),
+    "b200_lm_embed_bigram": (_I, [_P, _P, _F, _P, _I, _L, _L, _P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P, _F, _P, _P, _L, _I, _I,
+                                  _I, _P]),
+    "b200_lm_close_rows": (_I, [_P, _L, _I, _P, _L, _P, _F, _P, _L, _P, _F, _P, _L, _P, _F, _P, _L, _P, _F, _P, _L, _P, _L, _I, _I,
+                                _P]),
+    "b200_lm_table_gate_bf16": (_I, [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _P]),
     "b200_lm_rope_table": (_I, [_P, _P, _P, _I, _I, _F, _P]),
     "b200_lm_norm_rows": (_I, [_P, _L, _P, _I, _P, _F, _F, _P, _L, _I, _P, _I, _I, _P, _I, _I, _P]),
     "b200_lm_latent_post": (_I, [_P, _L, _P, _P, _F, _P, _L, _P, _I, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P]),
@@ -124,11 +129,11 @@ LM_SIGNATURES = {
                                         _P, _F, _P, _L, _I, _I, _P]),
     "b200_lm_moe_group": (_I, [_P, _I, _I, _P, _L, _P, _P]),
     "b200_lm_gemm_rows": (_I, [_P, _L, _L, _P, _L, _L, _P, _P, _L, _L, _P, _L, _P, _I, _I, _I, _I, _I, _I, _F, _I,
-                               _I, _I, _P]),
+                               _I, _I, _P, _L, _P, _L, _P, _I, _P]),
     "b200_lm_argmax_rows": (_I, [_P, _L, _I, _P, _P, _I, _P]),
     "b200_lm_rows_to_bf16": (_I, [_P, _L, _P, _I, _P, _L, _I, _I, _I, _I, _P]),
     "b200_gemm_wt_f32_grouped": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _I, _I, _I, _P]),
-    "b200_gemm_wt_f32_heads": (_I, [_P, _L, _I, _I, _P, _L, _P, _L, _L, _I, _I, _I, _I, _P]),
+    "b200_gemm_wt_f32_heads": (_I, [_P, _L, _I, _I, _P, _L, _P, _L, _L, _I, _I, _I, _I, _I, _P]),
     "b200_lm_moe_tiles": (_I, [_P, _L, _P, _I, _I, _P, _I, _P, _P]),
     "b200_lm_moe_order": (_I, [_P, _L, _P, _I, _P, _P]),
     "b200_lm_rows_scatter": (_I, [_P, _L, _P, _P, _L, _I, _I, _P]),
@@ -142,16 +147,22 @@ LM_SIGNATURES = {
     "b200_lm_token_shift": (_I, [_P, _L, _P, _P, _L, _L, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P]),
     "b200_lm_qkv_post": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _F, _I, _F, _I, _P,
                               _P, _L, _P, _L, _I, _P]),
-    "b200_lm_head_qkv_post": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _F, _I, _P]),
-    "b200_lm_sink_attention": (_I, [_P, _L, _P, _I, _L, _L, _P, _P, _P, _L, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P, _I, _I,
+    "b200_lm_head_qkv_post": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _F, _I, _I, _P]),
+    "b200_lm_sink_attention": (_I, [_P, _L, _P, _I, _L, _L, _P, _P, _P, _L, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _F, _P, _I, _I,
                                     _P]),
     "b200_lm_linear_state": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F,
                                   _P, _P, _L, _P, _P, _P, _L, _I, _I, _P, _P, _L, _P, _P, _I, _I, _P, _I, _I, _P]),
     "b200_lm_heads_to_bf16": (_I, [_P, _L, _I, _I, _P, _I, _I, _P]),
-    "b200_lm_sink_softmax_bf16": (_I, [_P, _L, _P, _I, _P, _F, _I, _I, _I, _F, _I, _I, _I, _I, _P, _L, _I, _I, _P]),
+    "b200_lm_sink_softmax_bf16": (_I, [_P, _L, _P, _I, _P, _F, _I, _I, _I, _F, _I, _I, _I, _I, _F, _P, _L, _I, _I, _P]),
     "b200_lm_head_post": (_I, [_P, _L, _P, _L, _P, _I, _F, _I, _I, _I, _I, _I, _F, _P, _L, _I, _I, _P]),
     "b200_lm_glu_clamp": (_I, [_P, _L, _P, _L, _F, _F, _F, _F, _I, _P, _L, _I, _I, _P]),
     "b200_lm_glu_clamp_bf16": (_I, [_P, _L, _P, _L, _F, _F, _F, _F, _I, _P, _I, _I, _P, _I, _P]),
+    # csrc/recurrent_ops.cu
+    "b200_lm_gated_recurrence": (_I, [_P, _L, _I, _P, _P, _P, _F, _P, _L, _P, _L, _P, _L, _P, _I, _P, _P, _I, _P, _L, _P, _L, _I,
+                                      _I, _P, _P]),
+    "b200_lm_matrix_memory_scratch": (_L, [_I, _I, _I, _I, _I]),
+    "b200_lm_matrix_memory": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _F, _F, _P, _L, _P, _F, _P, _L, _P, _I, _P, _P, _I, _I,
+                                   _I, _P, _L, _P, _L, _P, _L, _I, _I, _P]),
 }
 SIGNATURES.update(LM_SIGNATURES)
 

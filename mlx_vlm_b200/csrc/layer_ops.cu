@@ -47,6 +47,213 @@ __global__ void embed_scale_kernel(const int* __restrict__ tok, const bf16* __re
   for (int i = threadIdx.x; i < W; i += blockDim.x) x[(long)t * W + i] = bf2f(emb[(long)id * W + i]) * scale;
 }
 
+// The same with a second table that is addressed by the token and the one before it: row (prev mul_prev + cur mul_cur) mod
+// buckets, or row `buckets` for a sequence's first token.  The token before a step's first one is kept in the slot (one
+// state number, the id's bits).  The row may also be kept a second time (a model that adds the embedding output again), and
+// normed in the same launch, as fp32 rows and as bf16 operand rows (a block per token: it has the row in shared memory).
+struct EmbedP {
+  const int* tok;
+  const bf16* emb; float scale;
+  const bf16* big; int buckets; long long mul_prev, mul_cur;
+  float* state; long slot_stride;
+  const int *slot, *pos, *first;
+  int single;                          // every sequence of the step is one token: the block also leaves the token in the slot
+  float *x, *keep;
+  const bf16* nw; float eps;           // first norm's weight (NULL: none)
+  float* xn; bf16* xb; long ldb;
+  int W, vocab;
+};
+__device__ __forceinline__ int clamp_id(int id, int n) { return id < 0 ? 0 : (id >= n ? n - 1 : id); }
+__global__ void embed_bigram_kernel(EmbedP p) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  __shared__ int s_row;
+  const int t = blockIdx.x, id = clamp_id(p.tok[t], p.vocab);
+  if (threadIdx.x == 0) {
+    int row = p.buckets;
+    float* st = p.state + (long)p.slot[t] * p.slot_stride;
+    if (p.pos[t] > 0) {
+      const int prev = p.first[t] == t ? __float_as_int(*st) : clamp_id(p.tok[t - 1], p.vocab);
+      long long r = ((long long)prev * p.mul_prev + (long long)id * p.mul_cur) % p.buckets;
+      row = (int)(r < 0 ? r + p.buckets : r);
+    }
+    s_row = row;
+    if (p.single) *st = __int_as_float(id);
+  }
+  __syncthreads();
+  const bf16* b = p.big + (long)s_row * p.W;
+  const bf16* e = p.emb + (long)id * p.W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+    const float v = fmaf(bf2f(e[i]), p.scale, bf2f(b[i]));
+    p.x[(long)t * p.W + i] = v;
+    if (p.keep) p.keep[(long)t * p.W + i] = v;
+    if (p.nw) sm[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (!p.nw) return;
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps);
+  for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+    const float v = sm[i] * inv * bf2f(p.nw[i]);
+    p.xn[(long)t * p.W + i] = v;
+    if (p.xb) p.xb[(long)t * p.ldb + i] = f2bf(v);
+  }
+  if (p.xb)
+    for (int i = p.W + threadIdx.x; i < p.ldb; i += blockDim.x) p.xb[(long)t * p.ldb + i] = f2bf(0.f);
+}
+__global__ void last_token_kernel(const int* __restrict__ tok, const int* __restrict__ seqs, int n_seq,
+                                  const int* __restrict__ slot, float* __restrict__ state, long slot_stride, int vocab) {
+  const int g = blockIdx.x * blockDim.x + threadIdx.x;
+  if (g >= n_seq) return;
+  const int last = seqs[2 * g] + seqs[2 * g + 1] - 1;
+  state[(long)slot[last] * slot_stride] = __int_as_float(clamp_id(tok[last], vocab));
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// The residual update of up to three branches, some of them normed, and the norm that follows it, a block per row:
+//   x += sum_b mult_b N_b(y_b) [+ extra],   N_b(y) = y / sqrt(mean(y^2) + eps) * w_b   (w_b NULL: y itself)
+//   out = N(x) with weight nw (NULL: none);  xb = bf16 operand rows of out, or, without nw, of x.
+constexpr int CL_MAX = 3;
+struct CloseP {
+  float* x; long ldx;
+  int nb;
+  const float* y[CL_MAX]; long ldy[CL_MAX];
+  const bf16* w[CL_MAX];
+  float mult[CL_MAX];
+  const float* extra; long lde;
+  const bf16* nw; float eps;
+  float* out; long ldo;
+  bf16* xb; long ldb;
+  int N;
+};
+template <int V>
+struct RowVec { float v[V]; };
+template <int V>
+__device__ __forceinline__ RowVec<V> ld_vec(const float* p) {
+  RowVec<V> r;
+  if constexpr (V == 4) { const float4 a = *reinterpret_cast<const float4*>(p); r.v[0] = a.x; r.v[1] = a.y; r.v[2] = a.z; r.v[3] = a.w; }
+  else r.v[0] = *p;
+  return r;
+}
+template <int V>
+__device__ __forceinline__ void st_vec(float* p, const RowVec<V>& r) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  else *p = r.v[0];
+}
+template <int V>
+__device__ __forceinline__ RowVec<V> ld_vec(const bf16* p) {
+  RowVec<V> r;
+  if constexpr (V == 4) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&a.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&a.y);
+    r.v[0] = __low2float(lo); r.v[1] = __high2float(lo); r.v[2] = __low2float(hi); r.v[3] = __high2float(hi);
+  } else r.v[0] = bf2f(*p);
+  return r;
+}
+template <int V>
+__device__ __forceinline__ void st_vec(bf16* p, const RowVec<V>& r) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(r.v[0], r.v[1]), hi = __floats2bfloat162_rn(r.v[2], r.v[3]);
+    uint2 a;
+    a.x = *reinterpret_cast<const unsigned*>(&lo);
+    a.y = *reinterpret_cast<const unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(p) = a;
+  } else *p = f2bf(r.v[0]);
+}
+template <int V>
+__global__ void close_rows_kernel(CloseP p) {
+  extern __shared__ __align__(16) float row[];       // N: the updated row
+  __shared__ float red[CL_MAX][32];
+  const long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  float f[CL_MAX];
+  bool any = false;
+#pragma unroll
+  for (int b = 0; b < CL_MAX; ++b) {
+    f[b] = b < p.nb ? p.mult[b] : 0.f;
+    if (b < p.nb && p.w[b]) {
+      any = true;
+      float ss = 0.f;
+      const float* y = p.y[b] + t * p.ldy[b];
+      for (int i = threadIdx.x * V; i < p.N; i += blockDim.x * V) {
+        const RowVec<V> a = ld_vec<V>(y + i);
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss = fmaf(a.v[j], a.v[j], ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) red[b][warp] = ss;
+    }
+  }
+  if (any) {
+    __syncthreads();
+#pragma unroll
+    for (int b = 0; b < CL_MAX; ++b)
+      if (b < p.nb && p.w[b]) {
+        float tot = 0.f;
+        for (int i = 0; i < nw; ++i) tot += red[b][i];           // same order in every thread
+        f[b] /= sqrtf(tot / (float)p.N + p.eps);
+      }
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < p.N; i += blockDim.x * V) {
+    RowVec<V> x = ld_vec<V>(p.x + t * p.ldx + i);
+#pragma unroll
+    for (int b = 0; b < CL_MAX; ++b)
+      if (b < p.nb) {
+        const RowVec<V> a = ld_vec<V>(p.y[b] + t * p.ldy[b] + i);
+        if (p.w[b]) {
+          const RowVec<V> w = ld_vec<V>(p.w[b] + i);
+#pragma unroll
+          for (int j = 0; j < V; ++j) x.v[j] = fmaf(a.v[j] * f[b], w.v[j], x.v[j]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < V; ++j) x.v[j] = fmaf(a.v[j], f[b], x.v[j]);
+        }
+      }
+    if (p.extra) {
+      const RowVec<V> a = ld_vec<V>(p.extra + t * p.lde + i);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x.v[j] += a.v[j];
+    }
+    if (p.nb || p.extra) st_vec<V>(p.x + t * p.ldx + i, x);
+    if (p.nw) {
+      st_vec<V>(row + i, x);                     // read again by this thread only
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss = fmaf(x.v[j], x.v[j], ss);
+    } else if (p.xb) {
+      st_vec<V>(p.xb + t * p.ldb + i, x);
+    }
+  }
+  if (p.nw) {
+    const float inv = 1.0f / sqrtf(block_sum(ss, red[0]) / (float)p.N + p.eps);
+    for (int i = threadIdx.x * V; i < p.N; i += blockDim.x * V) {
+      RowVec<V> x = ld_vec<V>(row + i);
+      const RowVec<V> w = ld_vec<V>(p.nw + i);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x.v[j] = x.v[j] * inv * w.v[j];
+      if (p.out) st_vec<V>(p.out + t * p.ldo + i, x);
+      if (p.xb) st_vec<V>(p.xb + t * p.ldb + i, x);
+    }
+  }
+  if (p.xb)
+    for (long i = p.N + threadIdx.x; i < p.ldb; i += blockDim.x) p.xb[t * p.ldb + i] = f2bf(0.f);
+}
+
+// out[t][i] = gelu(z[t][i]) * table[tok[t]][i] as bf16 operand rows of ldo >= n columns (zero padding)
+__global__ void table_gate_bf16_kernel(const float* __restrict__ z, long ldz, const bf16* __restrict__ table, long ld_table,
+                                       int table_rows, const int* __restrict__ tok, bf16* __restrict__ out, int n, int ldo) {
+  const long t = blockIdx.x;
+  const bf16* e = table + (long)clamp_id(tok[t], table_rows) * ld_table;
+  for (int i = threadIdx.x; i < ldo; i += blockDim.x) {
+    float v = 0.f;
+    if (i < n) {
+      const float a = z[t * ldz + i];
+      v = a / (1.0f + expf(-1.5957691216057308f * (a + 0.044715f * a * a * a))) * bf2f(e[i]);
+    }
+    out[t * ldo + i] = f2bf(v);
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------
 // rotary table: cs[t][i] = amp * (cos, sin)(pos[t] * inv_freq[i]) with the angle in double precision (amp: the
 // amplitude that a frequency scaling puts on both, 1 without one)
@@ -548,7 +755,11 @@ struct GemmRowsP {
   int epi; float epi_param;              // 0 none, 1 relu^2, 2 param * tanh(v / param), 3 added to the output, 4 v * param, 5 gelu
   int round_x;
   int compact, n_batch;                  // compact: blockIdx.z counts the batches that HAVE rows (count[b] > 0) —
-};                                       // a decode step launches top x rows slices, not one per expert
+                                         // a decode step launches top x rows slices, not one per expert
+  const float* X2; long ldx2;            // != NULL (no batches, no lists): the rows multiplied are X + X2
+  const bf16* aux; long ld_aux;          // epi 6: the product passes the tanh form of gelu and is multiplied by
+  const int* aux_row; int aux_rows;      // aux[aux_row[output row]][n] (a table of aux_rows rows)
+};
 // the z-th batch with rows, or -1 (whole block; the counts are read 32 at a time, not one after the other)
 __device__ __forceinline__ int nth_active(const int* __restrict__ count, int n_batch, int z) {
   __shared__ int s_found;
@@ -577,6 +788,15 @@ __device__ __forceinline__ float gemm_epi(float v, int epi, float param) {
   if (epi == 4) return v * param;
   if (epi == 5) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));    // the exact gelu
   return v;
+}
+// epi 6: 0.5 v (1 + tanh(sqrt(2 / pi) (v + 0.044715 v^3))) = v sigmoid(2 sqrt(2 / pi) (...)), times a table's entry
+__device__ __forceinline__ float gelu_tanh(float v) {
+  return v / (1.0f + expf(-1.5957691216057308f * (v + 0.044715f * v * v * v)));
+}
+__device__ __forceinline__ float table_gate(const GemmRowsP& p, int row, int n, float v) {
+  int id = p.aux_row[row];
+  id = id < 0 ? 0 : (id >= p.aux_rows ? p.aux_rows - 1 : id);
+  return gelu_tanh(v) * bf2f(p.aux[(long)id * p.ld_aux + n]);
 }
 // epi 3: the product is added to what the output row holds (a residual stream that accumulates in place)
 __device__ __forceinline__ void gemm_store(float* y, float v, int epi, float param) {
@@ -615,7 +835,7 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(GemmRowsP p) {
       for (int j = 0; j < 4; ++j) {
         const int k = k0 + kk + j;
         float v = 0.f;
-        if (xr >= 0 && k < p.K) { v = X[(long)xr * p.ldx + k]; if (p.round_x) v = rbf(v); }
+        if (xr >= 0 && k < p.K) { v = X[(long)xr * p.ldx + k]; if (p.X2) v += p.X2[(long)xr * p.ldx2 + k]; if (p.round_x) v = rbf(v); }
         As[kk + j][r] = v;
       }
       const int n = n0 + r;
@@ -651,6 +871,7 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(GemmRowsP p) {
       if (n >= p.N) continue;
       float v = acc[i][j];
       if (p.bias) v += bf2f(p.bias[n]);
+      if (p.epi == 6) v = table_gate(p, yr, n, v);
       gemm_store(&Y[(long)yr * p.ldy + n], v, p.epi, p.epi_param);
     }
   }
@@ -687,14 +908,18 @@ __global__ void __launch_bounds__(256) gemm_skinny_kernel(GemmRowsP p) {
       for (int i = 0; i < GS_R; ++i)
         if (xr[i] >= 0) {
           float v = X[(long)xr[i] * p.ldx + k];
+          if (p.X2) v += p.X2[(long)xr[i] * p.ldx2 + k];
           if (p.round_x) v = rbf(v);
           acc[i] = fmaf(v, wv, acc[i]);
         }
     }
 #pragma unroll
     for (int i = 0; i < GS_R; ++i) {
-      const float v = warp_sum(acc[i]);
-      if (lane == 0 && yr[i] >= 0) gemm_store(&Y[(long)yr[i] * p.ldy + n], v + bias, p.epi, p.epi_param);
+      float v = warp_sum(acc[i]) + bias;
+      if (lane == 0 && yr[i] >= 0) {
+        if (p.epi == 6) v = table_gate(p, yr[i], n, v);
+        gemm_store(&Y[(long)yr[i] * p.ldy + n], v, p.epi, p.epi_param);
+      }
     }
   }
 }
@@ -737,6 +962,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemm_skinny_vec_kernel(GemmRows
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (xrow[i] >= 0) {
         v = *reinterpret_cast<const float4*>(X + (long)xrow[i] * p.ldx + k0 + k);
+        if (p.X2) {
+          const float4 u = *reinterpret_cast<const float4*>(p.X2 + (long)xrow[i] * p.ldx2 + k0 + k);
+          v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+        }
         if (p.round_x) { v.x = rbf(v.x); v.y = rbf(v.y); v.z = rbf(v.z); v.w = rbf(v.w); }
       }
       *reinterpret_cast<float4*>(&xs[i][k]) = v;
@@ -775,8 +1004,11 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemm_skinny_vec_kernel(GemmRows
     const float bias = (p.bias && n < p.N) ? bf2f(p.bias[n]) : 0.f;
 #pragma unroll
     for (int i = 0; i < MR; ++i) {
-      const float v = warp_sum(acc[r][i]);
-      if (lane == 0 && n < p.N && yrow[i] >= 0) gemm_store(&Y[(long)yrow[i] * p.ldy + n], v + bias, p.epi, p.epi_param);
+      float v = warp_sum(acc[r][i]) + bias;
+      if (lane == 0 && n < p.N && yrow[i] >= 0) {
+        if (p.epi == 6) v = table_gate(p, yrow[i], n, v);
+        gemm_store(&Y[(long)yrow[i] * p.ldy + n], v, p.epi, p.epi_param);
+      }
     }
   }
 }
@@ -949,6 +1181,10 @@ __global__ void __launch_bounds__(256) gemm_skinny_blk_kernel(GemmRowsP p) {
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (xrow[i] >= 0) {
         v = *reinterpret_cast<const float4*>(X + (long)xrow[i] * p.ldx + k0 + kk);
+        if (p.X2) {
+          const float4 u = *reinterpret_cast<const float4*>(p.X2 + (long)xrow[i] * p.ldx2 + k0 + kk);
+          v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+        }
         if (p.round_x) { v.x = rbf(v.x); v.y = rbf(v.y); v.z = rbf(v.z); v.w = rbf(v.w); }
       }
       *reinterpret_cast<float4*>(&xs[i][kk]) = v;
@@ -985,6 +1221,7 @@ __global__ void __launch_bounds__(256) gemm_skinny_blk_kernel(GemmRowsP p) {
     for (int w = 0; w < 8; ++w) v += red[w][r][i];
     if (n < p.N && yrow[i] >= 0) {
       if (p.bias) v += bf2f(p.bias[n]);
+      if (p.epi == 6) v = table_gate(p, yrow[i], n, v);
       gemm_store(&(p.Y + (long)b * p.yb)[(long)yrow[i] * p.ldy + n], v, p.epi, p.epi_param);
     }
   }
@@ -1052,6 +1289,55 @@ extern "C" {
 int b200_lm_embed(const int* tokens, const void* embed, float scale, float* x, int T, int W, int vocab, void* st) {
   B200_REQUIRE(tokens && embed && x && T > 0 && W > 0, "lm_embed: bad argument");
   embed_scale_kernel<<<T, 256, 0, (cudaStream_t)st>>>(tokens, (const bf16*)embed, scale, x, W, vocab);
+  B200_CHECK_LAUNCH();
+  return B200_OK;
+}
+
+int b200_lm_embed_bigram(const int* tokens, const void* embed, float scale, const void* bigram, int buckets, long mul_prev,
+                         long mul_cur, float* state, long slot_stride, const int* slot, const int* pos, const int* first,
+                         const int* seqs, int n_seq, int single, float* x, float* keep, const void* norm_w, float eps, float* xn,
+                         void* xb, long ldb, int T, int W, int vocab, void* st) {
+  B200_REQUIRE(tokens && embed && bigram && state && slot && pos && first && seqs && x && T > 0 && W > 0 && n_seq > 0 && buckets > 0,
+               "lm_embed_bigram: bad argument");
+  B200_REQUIRE(!norm_w || (xn && W <= 12000 && (!xb || ldb >= W)), "lm_embed_bigram: rows of %d numbers and their norm", W);
+  EmbedP p{tokens, (const bf16*)embed, scale, (const bf16*)bigram, buckets, mul_prev, mul_cur, state, slot_stride, slot, pos, first,
+           single, x, keep, (const bf16*)norm_w, eps, xn, (bf16*)xb, ldb, W, vocab};
+  embed_bigram_kernel<<<T, T < 64 ? 1024 : 256, norm_w ? W * sizeof(float) : 0, (cudaStream_t)st>>>(p);
+  B200_CHECK_LAUNCH();
+  if (!single) {
+    last_token_kernel<<<cdiv(n_seq, 128), 128, 0, (cudaStream_t)st>>>(tokens, seqs, n_seq, slot, state, slot_stride, vocab);
+    B200_CHECK_LAUNCH();
+  }
+  return B200_OK;
+}
+
+int b200_lm_close_rows(float* x, long ldx, int nb, const float* y0, long ldy0, const void* w0, float m0, const float* y1, long ldy1,
+                       const void* w1, float m1, const float* y2, long ldy2, const void* w2, float m2, const float* extra,
+                       long lde, const void* norm_w, float eps, float* out, long ldo, void* xb, long ldb, int T, int N, void* st) {
+  B200_REQUIRE(x && T > 0 && N > 0 && nb >= 0 && nb <= CL_MAX, "lm_close_rows: bad argument");
+  B200_REQUIRE((nb < 1 || y0) && (nb < 2 || y1) && (nb < 3 || y2), "lm_close_rows: %d branches", nb);
+  B200_REQUIRE((!norm_w || out || xb) && (!xb || ldb >= N), "lm_close_rows: the norm needs somewhere to go");
+  B200_REQUIRE(N <= 12000, "lm_close_rows: rows of %d numbers do not fit shared memory", N);
+  CloseP p{x, ldx, nb, {y0, y1, y2}, {ldy0, ldy1, ldy2}, {(const bf16*)w0, (const bf16*)w1, (const bf16*)w2}, {m0, m1, m2},
+           extra, lde, (const bf16*)norm_w, eps, out, ldo, (bf16*)xb, ldb, N};
+  uintptr_t al = (uintptr_t)x | (uintptr_t)extra | (uintptr_t)out | ((uintptr_t)norm_w << 1) | ((uintptr_t)xb << 1);
+  long ld = ldx | lde | ldo | ldb | N;
+  for (int b = 0; b < nb; ++b) { al |= (uintptr_t)p.y[b] | ((uintptr_t)p.w[b] << 1); ld |= p.ldy[b]; }
+  const bool vec = (al & 15) == 0 && (ld & 3) == 0;
+  const int per = vec ? cdiv(N, 4) : N;
+  int threads = T < 64 ? (per >= 1024 ? 1024 : cdiv(per, 32) * 32) : (per >= 256 ? 256 : cdiv(per, 32) * 32);
+  const size_t smem = norm_w ? (size_t)N * sizeof(float) : 0;
+  if (vec) close_rows_kernel<4><<<T, threads, smem, (cudaStream_t)st>>>(p);
+  else close_rows_kernel<1><<<T, threads, smem, (cudaStream_t)st>>>(p);
+  B200_CHECK_LAUNCH();
+  return B200_OK;
+}
+
+int b200_lm_table_gate_bf16(const float* z, long ldz, const void* table, long ld_table, int table_rows, const int* tokens, void* out,
+                            int n, int ldo, int T, void* st) {
+  B200_REQUIRE(z && table && tokens && out && T > 0 && n > 0 && ldo >= n && table_rows > 0, "lm_table_gate_bf16: bad argument");
+  table_gate_bf16_kernel<<<T, ldo >= 256 ? 256 : cdiv(ldo, 32) * 32, 0, (cudaStream_t)st>>>(z, ldz, (const bf16*)table, ld_table, table_rows,
+                                                                                           tokens, (bf16*)out, n, ldo);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }
@@ -1198,17 +1484,20 @@ int b200_lm_moe_group(const int* idx, int n_entries, int E, int* list, long list
 
 int b200_lm_gemm_rows(const float* X, long ldx, long xb, const void* W, long ldw, long wb, const void* bias, float* Y,
                       long ldy, long yb, const int* list, long list_stride, const int* count, int x_div, int M, int N,
-                      int K, int batch, int epi, float epi_param, int round_x, int skinny, int compact, void* st) {
+                      int K, int batch, int epi, float epi_param, int round_x, int skinny, int compact, const float* X2, long ldx2,
+                      const void* aux, long ld_aux, const int* aux_row, int aux_rows, void* st) {
   B200_REQUIRE(X && W && Y && M > 0 && N > 0 && K > 0 && batch > 0, "lm_gemm_rows: bad argument");
   B200_REQUIRE((list == nullptr) == (count == nullptr), "lm_gemm_rows: a row list needs its counts");
+  B200_REQUIRE(!X2 || (batch == 1 && !list), "lm_gemm_rows: a second addend goes with one plain product");
+  B200_REQUIRE(epi != 6 || (aux && aux_row && aux_rows > 0 && batch == 1 && !list), "lm_gemm_rows: the gated epilogue needs its table and one plain product");
   GemmRowsP p{X, ldx, xb, (const bf16*)W, ldw, wb, (const bf16*)bias, Y, ldy, yb, list, list_stride, count,
-              x_div > 0 ? x_div : 1, M, N, K, epi, epi_param, round_x, 0, batch};
+              x_div > 0 ? x_div : 1, M, N, K, epi, epi_param, round_x, 0, batch, X2, ldx2, (const bf16*)aux, ld_aux, aux_row, aux_rows};
   if (skinny && count && compact > 0 && compact < batch) {   // at most `compact` batches can have rows
     p.compact = 1;
     batch = compact;
   }
   const bool vec = K % 8 == 0 && ldw % 8 == 0 && wb % 8 == 0 && ldx % 4 == 0 && xb % 4 == 0 &&
-                   ((uintptr_t)W & 15) == 0 && ((uintptr_t)X & 15) == 0;
+                   ((uintptr_t)W & 15) == 0 && ((uintptr_t)X & 15) == 0 && (!X2 || (ldx2 % 4 == 0 && ((uintptr_t)X2 & 15) == 0));
   if (skinny && vec && M <= 16) {
     dim3 grid(cdiv(N, GV_WARPS * GV_R), 1, batch);
     const cudaStream_t cs = (cudaStream_t)st;

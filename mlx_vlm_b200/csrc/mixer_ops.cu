@@ -245,6 +245,7 @@ struct HeadQkvP {
   int H, G, dim, vdim, rot_dims, pairs;
   const bf16 *qn_w, *kn_w;         // [dim] or NULL
   float eps;
+  int unit;                        // the norms of queries and keys have no weight (qn_w, kn_w NULL)
 };
 template <typename CT>
 __global__ void head_qkv_post_kernel(HeadQkvP<CT> p) {
@@ -265,13 +266,14 @@ __global__ void head_qkv_post_kernel(HeadQkvP<CT> p) {
   const float* x = query ? q : p.K + (long)t * p.ldk + (long)h * p.dim;
   const bf16* w = query ? p.qn_w : p.kn_w;
   CT* kd = row + (long)h * p.dim;
+  const bool norm = w || p.unit;
   float inv = 1.f;
-  if (w) {
+  if (norm) {                      // the rotation keeps the sum of squares: a norm after it is the same as one before it
     float ss = 0.f;
     for (int i = lane; i < p.dim; i += 32) ss = fmaf(x[i], x[i], ss);
     inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);           // (also: every lane has read the row before one writes)
   }
-  auto in = [&](int i) { return w ? x[i] * inv * bf2f(w[i]) : x[i]; };
+  auto in = [&](int i) { return w ? x[i] * inv * bf2f(w[i]) : (norm ? x[i] * inv : x[i]); };
   auto put = [&](int i, float v) { if (query) q[i] = v; else st_row(kd + i, v); };
   for (int e = lane; e < half + p.dim - p.rot_dims; e += 32) {         // a lane reads and writes both numbers of its pair
     if (e >= half) { const int i = e + half; put(i, in(i)); continue; }
@@ -306,6 +308,7 @@ struct SinkAttnP {
   float bias_exp;                  // > 0: slope_h (query position - key position) is taken off the score of head h,
                                    // slope_h = 2^(-bias_exp (h + 1) / H)
   int unit_sink;                   // the denominator also holds exp(0) = 1 (a sink logit of zero, no tensor)
+  float softcap;                   // > 0: a score s becomes softcap tanh(s / softcap), before the distance bias
 };
 template <typename CT>
 __global__ void sink_attention_kernel(SinkAttnP<CT> p) {
@@ -393,7 +396,9 @@ __global__ void sink_attention_kernel(SinkAttnP<CT> p) {
       } else {
         for (int i = 0; i < dim; ++i) a = fmaf(qr[i], kr[i], a);
       }
-      s = a * p.scale - slope * (float)(ps - (k0 + lane));
+      s = a * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      s -= slope * (float)(ps - (k0 + lane));
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);       // nothing seen yet: exp(-inf) = 0
@@ -1371,9 +1376,9 @@ __global__ void heads_to_bf16_kernel(const float* __restrict__ q, long ldq, int 
   const float* x = q + (long)t * ldq + r * dim;
   for (int k = threadIdx.x; k < Kp; k += blockDim.x) out[(long)i * Kp + k] = f2bf(k < dim ? x[k] : 0.f);
 }
-__global__ void sink_softmax_bf16_kernel(const float* __restrict__ S, long lds, const int* __restrict__ pos, int rep,
+__global__ void sink_softmax_bf16_kernel(float* __restrict__ S, long lds, const int* __restrict__ pos, int rep,
                                          const bf16* __restrict__ sink, float scale, int chunk, int window, int key0,
-                                         float bias_exp, int head0, int H, int unit_sink, int split,
+                                         float bias_exp, int head0, int H, int unit_sink, int split, float softcap,
                                          bf16* __restrict__ P, long ldp, int Sp) {
   __shared__ float red[32];
   const long r = blockIdx.x;
@@ -1382,12 +1387,15 @@ __global__ void sink_softmax_bf16_kernel(const float* __restrict__ S, long lds, 
   if (chunk > 0) lo = max(lo, (ps / chunk) * chunk);
   if (window > 0) lo = max(lo, ps - window + 1);
   const int j0 = lo - key0, j1 = ps - key0;            // visible columns j0 .. j1
-  const float* s = S + r * lds;
+  float* s = S + r * lds;
   const float sk = sink ? bf2f(sink[r % rep]) : (unit_sink ? 0.f : -INFINITY);
   const float slope = bias_exp > 0.f ? exp2f(-bias_exp * (float)(head0 + (int)(r % rep) + 1) / (float)H) : 0.f;
   // the score of column j: scale s_j - slope (distance to the query); j1 - j is that distance
-  auto sc = [&](int j) { return s[j] * scale - slope * (float)(j1 - j); };
+  const float mul = softcap > 0.f ? 1.f : scale;
+  auto sc = [&](int j) { return s[j] * mul - slope * (float)(j1 - j); };
   float m = sk;
+  if (softcap > 0.f)                 // the scaled and capped score is left in place: the thread that made it reads it again
+    for (int j = j0 + threadIdx.x; j <= j1; j += blockDim.x) s[j] = softcap * tanhf(s[j] * scale / softcap);
   for (int j = j0 + threadIdx.x; j <= j1; j += blockDim.x) m = fmaxf(m, sc(j));
   m = warp_max(m);
   __syncthreads();
@@ -1495,19 +1503,20 @@ int b200_lm_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* 
 
 int b200_lm_head_qkv_post(float* Q, long ldq, const float* K, long ldk, const float* V, long ldv, void* cache, int cache_bf16,
                           long slot_stride, long tok_stride, const int* slot, const int* pos, const float* cs, int H, int G,
-                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int T,
-                          void* st) {
+                          int dim, int vdim, int rot_dims, int pairs, const void* qn_w, const void* kn_w, float eps, int unit,
+                          int T, void* st) {
   B200_REQUIRE(Q && K && V && cache && slot && pos && T > 0 && H > 0 && G > 0, "lm_head_qkv_post: bad argument");
   B200_REQUIRE(rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || cs), "lm_head_qkv_post: rotated dims %d of %d", rot_dims, dim);
+  B200_REQUIRE(!unit || (!qn_w && !kn_w), "lm_head_qkv_post: a norm with a weight, or without one, not both");
   const int warps = T < 64 ? 2 : 8;            // few tokens: smaller blocks, so that the heads of a token spread over the SMs
   const dim3 grid(T, cdiv(H + 2 * G, warps));
   if (cache_bf16) {
     HeadQkvP<bf16> p{Q, ldq, K, ldk, V, ldv, (bf16*)cache, slot_stride, tok_stride, slot, pos, (const float2*)cs, H, G, dim, vdim,
-                     rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps};
+                     rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps, unit};
     head_qkv_post_kernel<bf16><<<grid, warps * 32, 0, (cudaStream_t)st>>>(p);
   } else {
     HeadQkvP<float> p{Q, ldq, K, ldk, V, ldv, (float*)cache, slot_stride, tok_stride, slot, pos, (const float2*)cs, H, G, dim, vdim,
-                      rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps};
+                      rot_dims, pairs, (const bf16*)qn_w, (const bf16*)kn_w, eps, unit};
     head_qkv_post_kernel<float><<<grid, warps * 32, 0, (cudaStream_t)st>>>(p);
   }
   B200_CHECK_LAUNCH();
@@ -1516,8 +1525,8 @@ int b200_lm_head_qkv_post(float* Q, long ldq, const float* K, long ldk, const fl
 
 int b200_lm_sink_attention(const float* q, long ldq, const void* cache, int cache_bf16, long slot_stride, long tok_stride,
                            const int* slot, const int* pos, float* out, long ldo, const void* sink, int H, int G,
-                           int dim, int vdim, float scale, int chunk, int window, float bias_exp, int unit_sink, float* part,
-                           int n_split, int T, void* st) {
+                           int dim, int vdim, float scale, int chunk, int window, float bias_exp, int unit_sink, float softcap,
+                           float* part, int n_split, int T, void* st) {
   B200_REQUIRE(q && cache && slot && pos && out && T > 0 && H > 0 && G > 0 && H % G == 0, "lm_sink_attention: bad argument");
   B200_REQUIRE(vdim <= 256, "lm_sink_attention: value size %d not supported", vdim);
   B200_REQUIRE(!(sink && unit_sink), "lm_sink_attention: a sink logit per head or the constant one, not both");
@@ -1531,13 +1540,13 @@ int b200_lm_sink_attention(const float* q, long ldq, const void* cache, int cach
     if (first_use_on_device(&g_sink_attr_bf16))
       B200_CUDA(cudaFuncSetAttribute(sink_attention_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     const int vec = dim % 8 == 0 && vdim % 8 == 0 && tok_stride % 8 == 0 && slot_stride % 8 == 0 && ((uintptr_t)cache & 15) == 0;
-    SinkAttnP<bf16> p{q, ldq, (const bf16*)cache, slot_stride, tok_stride, slot, pos, out, ldo, (const bf16*)sink, H, G, dim, vdim, scale, chunk, window, part, n_split, vec, bias_exp, unit_sink};
+    SinkAttnP<bf16> p{q, ldq, (const bf16*)cache, slot_stride, tok_stride, slot, pos, out, ldo, (const bf16*)sink, H, G, dim, vdim, scale, chunk, window, part, n_split, vec, bias_exp, unit_sink, softcap};
     sink_attention_kernel<bf16><<<grid, nw * 32, smem, (cudaStream_t)st>>>(p);
   } else {
     if (first_use_on_device(&g_sink_attr_f32))
       B200_CUDA(cudaFuncSetAttribute(sink_attention_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     const int vec = dim % 4 == 0 && vdim % 4 == 0 && tok_stride % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)cache & 15) == 0;
-    SinkAttnP<float> p{q, ldq, (const float*)cache, slot_stride, tok_stride, slot, pos, out, ldo, (const bf16*)sink, H, G, dim, vdim, scale, chunk, window, part, n_split, vec, bias_exp, unit_sink};
+    SinkAttnP<float> p{q, ldq, (const float*)cache, slot_stride, tok_stride, slot, pos, out, ldo, (const bf16*)sink, H, G, dim, vdim, scale, chunk, window, part, n_split, vec, bias_exp, unit_sink, softcap};
     sink_attention_kernel<float><<<grid, nw * 32, smem, (cudaStream_t)st>>>(p);
   }
   B200_CHECK_LAUNCH();
@@ -1633,12 +1642,12 @@ int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int dim, void* out,
   return B200_OK;
 }
 
-int b200_lm_sink_softmax_bf16(const float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
-                              int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, void* P,
+int b200_lm_sink_softmax_bf16(float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
+                              int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, float softcap, void* P,
                               long ldp, int rows, int Sp, void* st) {
   B200_REQUIRE(S && pos && P && rows > 0 && rep > 0 && Sp > 0 && key0 >= 0, "lm_sink_softmax_bf16: bad argument");
   sink_softmax_bf16_kernel<<<rows, 256, 0, (cudaStream_t)st>>>(S, lds, pos, rep, (const bf16*)sink, scale, chunk, window,
-                                                                key0, bias_exp, head0, H > 0 ? H : 1, unit_sink, split, (bf16*)P, ldp, Sp);
+                                                                key0, bias_exp, head0, H > 0 ? H : 1, unit_sink, split, softcap, (bf16*)P, ldp, Sp);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }

@@ -93,7 +93,10 @@ class LayerEngine:
     def _forward(self, tokens, slot, pos, want, embeds, segments):
         c, ops = self.core, self.ops
         ctx = StepCtx(ops, slot, pos, self.pool, c.eps, segments)    # segments: the host's view of a prompt step
-        if embeds is not None:
+        ctx.tokens = tokens
+        if hasattr(c, "embed_rows"):      # a design whose embedding needs more of the step than the token ids
+            x = c.embed_rows(ctx, tokens)
+        elif embeds is not None:
             with torch.cuda.stream(self.stream):
                 x = embeds.to(torch.float32).reshape(-1, c.width).clone()
         else:

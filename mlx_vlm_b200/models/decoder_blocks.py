@@ -51,6 +51,17 @@ and, for layers that norm the SUM of a scaled stream and a branch (the sublayers
   feed-forwards  NORMED_SUM_FEEDFORWARDS["dense"]      -> GatedDense with relu on the gate
   layer          NormedSumLayer: x = LN(a * x + mixer(x)); x = LN(a * x + ff(x)), layer norms with a bias
 
+and, for plain pre-norm layers with an input that a token brings to every layer:
+
+  mixers         PRENORM_MIXERS["parallel"] -> PairedMixer: a GroupedAttention (biases, unit-mean-square queries and keys,
+                                               soft-capped scores, a window, one in the denominator) beside a MatrixMemory
+                                               (exponential gates); half the sum of their outputs, each with a norm of its own
+                 PRENORM_MIXERS["rglru"]    -> GatedRecurrence (a gated linear recurrence per channel behind a convolution,
+                                               times a gelu branch)
+  feed-forwards  PRENORM_FEEDFORWARDS["dense"] -> GatedDense with silu on the gate
+  token input    TokenSide: x += N(W_proj (gelu(W_gate x) * the layer's slice of a table's row of the token))
+  layer          PreNormLayer: x += mixer(N1(x)); x += ff(N2(x)); x += the token input
+
 A block declares `manifest(prefix)` (packed name, shape) and `pack(prefix, checkpoint tensors, arena)`; the model
 packs all blocks into ONE device arena (the layout the other models of this package use).  `forward(ctx, x)`
 enqueues the block's kernels; `ctx` carries the per-token slot / position arrays of the step and the cache pool,
@@ -64,8 +75,8 @@ from typing import Dict, List, Optional
 import torch
 
 from .._native import B200Error as _B200Error
-from .layer_ops import (ACT_GELU, ACT_TANH, EPI_GELU, EPI_RELU2, EPI_SOFTCAP, GELU_TANH_ALPHA, GELU_TANH_CUBIC, WAVELENGTH,
-                        LayerOps)
+from .layer_ops import (ACT_GELU, ACT_TANH, EPI_GELU, EPI_RELU2, EPI_SOFTCAP, EPI_TABLE_GATE, GELU_TANH_ALPHA, GELU_TANH_CUBIC,
+                        WAVELENGTH, LayerOps)
 
 
 @dataclass
@@ -81,6 +92,9 @@ class StepCtx:
     carry: Dict = field(default_factory=dict)     # what one layer of the step leaves for later ones (rows of the step)
     x_operand: Optional[torch.Tensor] = None      # bf16 operand rows of the residual stream, where the sublayers read the
                                                   # stream itself and the norm that closed the last one wrote them
+    tokens: Optional[torch.Tensor] = None         # (T,) int32 device: the token ids of the step
+    kv_base: int = 0                              # caching layers and state numbers of the slot that lie before those of the
+    state_base: int = 0                           # current RUN of a layer (a layer that runs several times keeps one set per run)
 
     def seq_tables(self):
         """(first (T,), seqs (G, 2), G): the sequences of the step for the mixers that walk them in order; without a
@@ -1054,12 +1068,15 @@ class GroupedAttention:
     """Softmax attention with `heads` query heads over `kv_heads` key/value heads (query head h reads key/value head
     h // (heads / kv_heads)), q, k, v one stacked product of the mixer's input.  Optional, each by a parameter:
       qk_norm     "whole" (or True): q and k are RMS-normed over their WHOLE projection (all heads at once) and weighted
-                  (`q.norm`, `k.norm`); "head": every head by itself, with one weight vector for all query (key) heads
+                  (`q.norm`, `k.norm`); "head": every head by itself, with one weight vector for all query (key)
+                  heads; "unit": every head by itself, without a weight
       rot         rotary on the first `rot.dims` numbers of every head, pairs (i, i + dims / 2) (rotation="half") or
                   (2i, 2i + 1) ("pairs"), frequencies rescaled by `rot.scaling`: the YaRN rule (factor, original, fast,
                   slow) or the rule by wavelength (factor, original, low, high)
       v_from_k    the values are the keys as projected, before norm and rotation: no value projection
       v_unit      every value head is divided by its root mean square; the cache holds it so
+      bias        the projections have biases (`q.b`, `k.b`, `v.b`)
+      softcap     a scaled score s becomes softcap tanh(s / softcap) (from the configuration's `softcap`)
       sink        "learned": a logit per head (`sink`) joins the softmax's denominator without a key or a value;
                   "unit": the denominator holds one more 1 (a sink logit of zero)
       q_temp      queries times 1 + coef ln(floor((p + 1) / every) + 1) at position p
@@ -1069,8 +1086,9 @@ class GroupedAttention:
                   step) and the later ones (`"blend"`: v <- (1 - lam) v + lam v_first, lam = `vmix`, after the value norm)."""
 
     def __init__(self, index: int, cfg: dict, width: int, qk_norm=False, v_unit: bool = False,
-                 sink: Optional[str] = None, bias_exp: float = 0.0, rotation: str = "half", v_from_k: bool = False):
-        self.index, self.W = index, width
+                 sink: Optional[str] = None, bias_exp: float = 0.0, rotation: str = "half", v_from_k: bool = False,
+                 bias: bool = False):
+        self.index, self.W, self.bias = index, width, bool(bias)
         self.H, self.dim = int(cfg["heads"]), int(cfg["dim"])
         self.G, self.vdim = int(cfg.get("kv_heads", self.H)), int(cfg.get("vdim", self.dim))
         if self.H % self.G:
@@ -1090,10 +1108,11 @@ class GroupedAttention:
         self.q_temp = None if not qt else (float(qt["coef"]), int(qt["every"]))
         if sink not in (None, "learned", "unit"):
             raise ValueError(f"layer {index}: sink {sink!r} (have None, 'learned', 'unit')")
-        if rotation not in ("half", "pairs") or qk_norm not in (False, True, "whole", "head"):
+        if rotation not in ("half", "pairs") or qk_norm not in (False, True, "whole", "head", "unit"):
             raise ValueError(f"layer {index}: rotation {rotation!r} (have 'half', 'pairs'), query/key norm {qk_norm!r}")
         self.qk_norm, self.v_unit, self.sink, self.bias_exp = bool(qk_norm), bool(v_unit), sink, float(bias_exp)
-        self.head_norm, self.pairs, self.v_from_k = qk_norm == "head", rotation == "pairs", bool(v_from_k)
+        self.head_norm, self.pairs, self.v_from_k = qk_norm in ("head", "unit"), rotation == "pairs", bool(v_from_k)
+        self.unit_norm, self.softcap = qk_norm == "unit", float(cfg.get("softcap") or 0.0)
         self.per_head = self.head_norm or self.pairs      # the step between projection and cache is the per-head one
         self.v_mix = bool(cfg.get("v_mix"))
         self.v_role: Optional[str] = None      # set by the model: "first" / "blend"
@@ -1103,14 +1122,23 @@ class GroupedAttention:
         if self.v_from_k and (self.vdim != self.dim or self.v_mix):
             raise ValueError(f"layer {index}: values that are the keys have the keys' size ({self.vdim} and {self.dim})")
         self.n_q, self.n_k, self.n_v = self.H * self.dim, self.G * self.dim, self.G * self.vdim
+        self.n_in, self.n_out = self.n_q + self.n_k + (0 if self.v_from_k else self.n_v), self.H * self.vdim
         self.kv_dim, self.state_floats = self.n_k + self.n_v, 0
         self.cache_index, self.state_off = -1, 0
         self.w: Dict[str, torch.Tensor] = {}
 
+    def in_parts(self):
+        """(checkpoint name, rows, has a bias) of the projections of the mixer's input, stacked in this order"""
+        return [("q", self.n_q, self.bias), ("k", self.n_k, self.bias)] + ([] if self.v_from_k else [("v", self.n_v, self.bias)])
+
+    def small(self):
+        return []            # (tensors beside the projections that a PairedMixer packs: none in the forms it uses)
+
     def manifest(self, p: str):
-        out = [(p + "qkv", (self.n_q + self.n_k + (0 if self.v_from_k else self.n_v), self.W)),
-               (p + "o", (self.W, self.H * self.vdim))]
-        if self.qk_norm:
+        out = [(p + "qkv", (self.n_in, self.W)), (p + "o", (self.W, self.n_out))]
+        if self.bias:
+            out.append((p + "qkv.b", (self.n_in,)))
+        if self.qk_norm and not self.unit_norm:
             out += [(p + "q.norm", (self.dim if self.head_norm else self.n_q,)),
                     (p + "k.norm", (self.dim if self.head_norm else self.n_k,))]
         if self.sink == "learned":
@@ -1120,9 +1148,11 @@ class GroupedAttention:
         return out
 
     def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
-        out = {p + "q": (self.n_q, self.W), p + "k": (self.n_k, self.W), p + "o": (self.W, self.H * self.vdim)}
-        if not self.v_from_k:
-            out[p + "v"] = (self.n_v, self.W)
+        out = {p + "o": (self.W, self.n_out)}
+        for n, rows, bias in self.in_parts():
+            out[p + n] = (rows, self.W)
+            if bias:
+                out[p + n + ".b"] = (rows,)
         out.update({n: s for n, s in self.manifest(p) if n in (p + "q.norm", p + "k.norm")})
         if self.sink == "learned":
             out[p + "sink"] = (self.H,)
@@ -1131,25 +1161,31 @@ class GroupedAttention:
         return out
 
     def pack(self, p: str, ck, view):
-        qkv = view(p + "qkv")
-        qkv[:self.n_q].copy_(ck[p + "q"])
-        qkv[self.n_q:self.n_q + self.n_k].copy_(ck[p + "k"])
-        if not self.v_from_k:
-            qkv[self.n_q + self.n_k:].copy_(ck[p + "v"])
+        r = 0
+        for n, rows, bias in self.in_parts():
+            view(p + "qkv")[r:r + rows].copy_(ck[p + n])
+            if bias:
+                view(p + "qkv.b")[r:r + rows].copy_(ck[p + n + ".b"])
+            r += rows
         for n, shape in self.manifest(p)[1:]:
-            view(n).copy_(ck[n].reshape(shape))
+            if n != p + "qkv.b":
+                view(n).copy_(ck[n].reshape(shape))
         self.bind(p, view)
 
     def bind(self, p: str, view):
         self.w = {n[len(p):]: view(n) for n, _ in self.manifest(p)}
 
     def forward(self, ctx: StepCtx, h: torch.Tensor) -> torch.Tensor:
-        ops, w, T = ctx.ops, self.w, h.shape[0]
+        D = ctx.ops.linear(h, self.w["qkv"], bias=self.w.get("qkv.b"), operand=ctx.x_operand)
+        return ctx.ops.linear(self.attend(ctx, D), self.w["o"])
+
+    def attend(self, ctx: StepCtx, D: torch.Tensor) -> torch.Tensor:
+        """D (T, n_in): the projected rows (scratch) -> the heads' outputs side by side (T, n_out)"""
+        ops, w, T = ctx.ops, self.w, D.shape[0]
         nq, nk, nv = self.n_q, self.n_k, self.n_v
-        D = ops.linear(h, w["qkv"], operand=ctx.x_operand)
         q, k = D[:, :nq], D[:, nq:nq + nk]
-        v = k if self.v_from_k else D[:, nq + nk:]
-        rows = ctx.pool.buf[self.cache_index][..., :self.kv_dim]
+        v = k if self.v_from_k else D[:, nq + nk:nq + nk + nv]
+        rows = ctx.pool.buf[ctx.kv_base + self.cache_index][..., :self.kv_dim]
         cs = ctx.rope(self.rot_base, self.rot_dims, self.rot_scaling)
         v_first = keep = None
         if self.v_role == "first":
@@ -1158,7 +1194,7 @@ class GroupedAttention:
             v_first = ctx.carry["v_first"]
         if self.per_head:
             ops.head_qkv_post(q, k, v, rows, ctx.slot, ctx.pos, cs, self.H, self.G, self.dim, self.vdim, self.rot_dims,
-                              q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps, pairs=self.pairs)
+                              q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps, pairs=self.pairs, unit=self.unit_norm)
         else:
             ops.qkv_post(q, k, v, rows, ctx.slot, ctx.pos, cs, self.H, self.G, self.dim, self.vdim, self.rot_dims,
                          q_norm=w.get("q.norm"), k_norm=w.get("k.norm"), eps=ctx.eps, v_unit=self.v_unit, q_temp=self.q_temp,
@@ -1179,7 +1215,7 @@ class GroupedAttention:
                 ops.tc_refused(e)
         if not done:
             self._attend_rows(ctx, q, rows, ctx.slot, ctx.pos, o, prompt=ctx.segments is not None)
-        return ops.linear(o, w["o"])
+        return o
 
     def _tc_portion(self, ops: LayerOps, n: int, rows) -> bool:
         return ops.tc_ok(n, self.dim, rows.stride(1)) and rows.stride(0) % 8 == 0
@@ -1189,7 +1225,7 @@ class GroupedAttention:
         keys of a query over several blocks"""
         ctx.ops.sink_attention(q, rows, slot, pos, o, self.w.get("sink"), self.H, self.G, self.dim, self.vdim, self.scale,
                                window=self.window, n_split=1 if prompt and q.shape[0] > 16 else None,
-                               bias_exp=self.bias_exp, unit_sink=self.sink == "unit")
+                               bias_exp=self.bias_exp, unit_sink=self.sink == "unit", softcap=self.softcap)
 
     def _attend_prompt(self, ctx: StepCtx, q, all_rows, slot_index: int, pos, o, p0: int, n: int):
         """A portion of a prompt (positions p0 .. p0 + n - 1 of one slot) as two tcgen05 products per key/value head:
@@ -1223,7 +1259,7 @@ class GroupedAttention:
                     P = ops.empty((mm * rep, 2 * Sp), torch.bfloat16)
                     ops.sink_softmax_bf16(sc, pos[b:b + mm], rep, None if sink is None else sink[g * rep:], self.scale, 0,
                                           self.window, key0, P, bias_exp=self.bias_exp, head0=g * rep, H=H,
-                                          unit_sink=self.sink == "unit", split=True)
+                                          unit_sink=self.sink == "unit", split=True, softcap=self.softcap)
                     og = ops.empty((mm * rep, dv))
                     ops.tc_gemm(P, vt, og, N_=dv, K=Sp, parts=2)
                     ops.head_post(og.view(mm, rep * dv), o[b:b + mm, g * rep * dv:(g + 1) * rep * dv], dv=dv)
@@ -1690,6 +1726,304 @@ class NormedSumLayer:
 
     def _close(self, ctx: StepCtx, x, y, norm: str):
         ctx.x_operand = ctx.ops.sum_norm_rows(y, x, self.w[norm], self.w[norm + ".b"], ctx.eps, keep=self.alpha, center=True)
+
+
+# ----------------------------------------------------------------------------------------------------------------
+# Plain pre-norm layers with an input that the token brings to every layer.  A mixer has `forward(ctx, h) -> branches
+# [(rows (T, width), norm weight or None, factor)]` of the residual update, `kv_dim` and `state_floats`; what a run of the
+# layer keeps in the slot begins at `ctx.kv_base` / `ctx.state_base`.
+def whole_vectors(n: int) -> int:
+    return (n + 3) // 4 * 4           # state spans start on 16-byte boundaries
+
+
+class MatrixMemory:
+    """Matrix memory with exponential gates (the mLSTM of Beck et al., "xLSTM: Extended Long Short-Term Memory").  q = W_q h
+    dim^-1/2, k = W_k h (`heads` x `dim`), v = W_v h (`heads` x `vdim`); per head a log input gate i = c tanh((W_i h + b_i) / c)
+    and a log forget gate f = logsigmoid(c tanh((W_f h + b_f) / c)), c = `gate_cap`.  With S (dim, vdim), n (dim) and the
+    running maximum m fp32 in the slot, all zero at position 0:  m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;
+    n likewise with k alone;  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6).  Every head's o is divided by its root mean square,
+    the heads side by side are multiplied by `norm` and sigmoid(W_g h), then W_o."""
+
+    def __init__(self, index: int, cfg: dict, width: int):
+        self.index, self.W = index, width
+        self.H, self.dim, self.cap = int(cfg["heads"]), int(cfg["dim"]), float(cfg["gate_cap"])
+        self.vdim = int(cfg.get("vdim", self.dim))
+        self.n_qk, self.n_v = self.H * self.dim, self.H * self.vdim
+        self.n_in, self.n_out = 2 * self.n_qk + 2 * self.n_v + 2 * self.H, self.n_v
+        self.kv_dim, self.state_floats = 0, whole_vectors(self.H * (self.dim * (self.vdim + 1) + 1))
+        self.cache_index, self.state_off = -1, 0
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def in_parts(self):
+        return [("q", self.n_qk, False), ("k", self.n_qk, False), ("v", self.n_v, False), ("g", self.n_v, False),
+                ("i", self.H, True), ("f", self.H, True)]
+
+    def small(self):
+        return [("norm", (self.n_v,))]
+
+    def mix(self, ctx: StepCtx, D: torch.Tensor, operand: bool = False) -> torch.Tensor:
+        """D (T, n_in): the projected rows -> the gated outputs (T, n_v), or (operand) their bf16 operand rows"""
+        a, b = self.n_qk, self.n_v
+        at = ctx.state_base + self.state_off
+        return ctx.ops.matrix_memory(D[:, :a], D[:, a:2 * a], D[:, 2 * a:2 * a + b], D[:, 2 * (a + b):2 * (a + b) + self.H],
+                                     D[:, 2 * (a + b) + self.H:self.n_in], D[:, 2 * a + b:2 * (a + b)], self.w["norm"],
+                                     ctx.pool.state[:, at:at + self.state_floats], ctx, H=self.H, dim=self.dim, vdim=self.vdim,
+                                     cap=self.cap, q_scale=float(self.dim) ** -0.5, eps=ctx.eps, operand=operand)
+
+
+class PairedMixer:
+    """An attention (`left`) and a matrix memory (`right`) that read the same input: half the sum of their outputs, each first
+    RMS-normed over the width with a weight of its own (`left.out`, `right.out`).  All their input projections are ONE product,
+    the norms, the factors and the sum belong to the residual update."""
+
+    def __init__(self, index: int, cfg: dict, width: int, left, right, factor: float = 0.5):
+        self.index, self.W, self.left, self.right, self.factor = index, width, left, right, float(factor)
+        self.n_in = (left.n_in + right.n_in + 7) // 8 * 8            # whole vectors per row; the rows beyond are zeros
+        self.kv_dim = left.kv_dim
+        left.cache_index, left.state_off, right.state_off = 0, 0, left.state_floats
+        self.state_floats = left.state_floats + right.state_floats
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def _sides(self):
+        return (("left.", self.left), ("right.", self.right))
+
+    def manifest(self, p: str):
+        out = [(p + "in", (self.n_in, self.W)), (p + "in.b", (self.n_in,))]
+        for s, m in self._sides():
+            out += [(p + s + "o", (self.W, m.n_out)), (p + s + "out", (self.W,))] + [(p + s + n, shape) for n, shape in m.small()]
+        return out
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        out = dict(self.manifest(p)[2:])
+        for s, m in self._sides():
+            for n, rows, bias in m.in_parts():
+                out[p + s + n] = (rows, self.W)
+                if bias:
+                    out[p + s + n + ".b"] = (rows,)
+        return out
+
+    def pack(self, p: str, ck, view):
+        w_in, b_in, r = view(p + "in"), view(p + "in.b"), 0
+        b_in.zero_()
+        for s, m in self._sides():
+            for n, rows, bias in m.in_parts():
+                w_in[r:r + rows].copy_(ck[p + s + n])
+                if bias:
+                    b_in[r:r + rows].copy_(ck[p + s + n + ".b"])
+                r += rows
+        w_in[r:].zero_()
+        for n, _ in self.manifest(p)[2:]:
+            view(n).copy_(ck[n])
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n[len(p):]: view(n) for n, _ in self.manifest(p)}
+        for s, m in self._sides():
+            m.w = {n: view(p + s + n) for n, _ in m.small()}
+
+    def forward(self, ctx: StepCtx, h: torch.Tensor) -> List[tuple]:
+        ops, w, T = ctx.ops, self.w, h.shape[0]
+        D = ops.linear(h, w["in"], bias=w["in.b"], operand=ctx.x_operand)
+        a, b = self.left.n_in, self.right.n_in
+        yl = ops.linear(self.left.attend(ctx, D[:, :a]), w["left.o"])
+        op = ops.takes_operand(T, w["right.o"])
+        r = self.right.mix(ctx, D[:, a:a + b], operand=op)
+        yr = ops.operand_linear(r, w["right.o"]) if op else ops.linear(r, w["right.o"])
+        return [(yl, w["left.out"], self.factor), (yr, w["right.out"], self.factor)]
+
+
+class GatedRecurrence:
+    """Griffin's recurrent block (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for Efficient
+    Language Models") with its real-gated linear recurrent unit, of `width` channels:  y = gelu(W_y h + b_y) (tanh form),
+    u = conv(W_x h + b_x) (causal, per channel, `conv` taps and a bias; the slot keeps the last taps - 1 inputs), in each of
+    `blocks` equal parts  r = sigmoid(R u + b_r), i = sigmoid(I u + b_i)  (square matrices);  log a = -decay r softplus(lam),
+    S <- a S + sqrt(1 - a^2) i u  (fp32 in the slot, zero at position 0);  output W_o (S y).
+    The gates' products read u in fp32 (two bf16 parts on the tensor cores): they enter the recurrence."""
+
+    def __init__(self, index: int, cfg: dict, width: int, decay: float = 8.0):
+        self.index, self.W, self.decay = index, width, float(decay)
+        self.n, self.blocks, self.taps = int(cfg["width"]), int(cfg["blocks"]), int(cfg.get("conv") or 1)
+        if self.n % self.blocks:
+            raise ValueError(f"layer {index}: {self.n} channels do not divide into {self.blocks} blocks")
+        self.bs = self.n // self.blocks
+        self.kv_dim = 0
+        self.conv_floats = max(self.taps - 1, 0) * self.n
+        self.state_floats = whole_vectors(self.conv_floats + self.n)
+        self.cache_index, self.state_off = -1, 0
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def manifest(self, p: str):
+        n, nb, bs = self.n, self.blocks, self.bs
+        return [(p + "yx", (2 * n, self.W)), (p + "yx.b", (2 * n,)), (p + "conv", (n, self.taps)), (p + "conv.b", (n,)),
+                (p + "gates", (nb, 2 * bs, bs)), (p + "ra.b", (n,)), (p + "ri.b", (n,)), (p + "lam", (n,)), (p + "o", (self.W, n))]
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        n, nb, bs = self.n, self.blocks, self.bs
+        out = {p + "conv": (n, self.taps), p + "conv.b": (n,), p + "lam": (n,), p + "o": (self.W, n)}
+        for s in ("y", "x"):
+            out.update({p + s: (n, self.W), p + s + ".b": (n,)})
+        for s in ("ra", "ri"):
+            out.update({p + s: (nb, bs, bs), p + s + ".b": (nb, bs)})
+        return out
+
+    def pack(self, p: str, ck, view):
+        for i, s in enumerate(("y", "x")):
+            view(p + "yx")[i * self.n:(i + 1) * self.n].copy_(ck[p + s])
+            view(p + "yx.b")[i * self.n:(i + 1) * self.n].copy_(ck[p + s + ".b"])
+        for i, s in enumerate(("ra", "ri")):         # both gates of a block are one product
+            view(p + "gates")[:, i * self.bs:(i + 1) * self.bs].copy_(ck[p + s])
+            view(p + s + ".b").copy_(ck[p + s + ".b"].reshape(-1))
+        for s in ("conv", "conv.b", "lam", "o"):
+            view(p + s).copy_(ck[p + s])
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n[len(p):]: view(n) for n, _ in self.manifest(p)}
+
+    def _gate_logits(self, ops: LayerOps, u: torch.Tensor) -> torch.Tensor:
+        """u (T, n) -> (T, 2 n): per block [r | i], without the biases"""
+        T, nb, bs, w = u.shape[0], self.blocks, self.bs, self.w["gates"]
+        G = ops.empty((T, 2 * self.n))
+        if ops.tc_ok(T, bs):
+            try:
+                if bs % 64 == 0:       # all blocks in ONE launch (inner sizes are whole k-blocks)
+                    us = ops.to_split(u.view(T * nb, bs), bs).view(T, 2 * self.n)
+                    ops.tc_gemm_heads(us, w, G, H=nb, N_=2 * bs, K=bs, x_cols=2 * self.n, x_group_cols=2 * bs, c_group_cols=2 * bs,
+                                      parts=2)
+                else:
+                    for b in range(nb):
+                        ops.linear(u[:, b * bs:(b + 1) * bs], w[b], out=G[:, 2 * b * bs:2 * (b + 1) * bs], exact_x=True)
+                return G
+            except _B200Error as e:
+                ops.tc_refused(e)
+        ops.gemm(u, w, G, M=T, N_=2 * bs, K=bs, xb=bs, ldw=bs, wb=2 * bs * bs, yb=2 * bs, batch=nb, exact_x=True)
+        return G
+
+    def forward(self, ctx: StepCtx, h: torch.Tensor) -> List[tuple]:
+        ops, w, T, n = ctx.ops, self.w, h.shape[0], self.n
+        at = ctx.state_base + self.state_off
+        D = ops.linear(h, w["yx"], bias=w["yx.b"], operand=ctx.x_operand)
+        u = ops.short_conv(D[:, n:], w["conv"], ctx.pool.state[:, at:at + self.conv_floats], ctx, bias=w["conv.b"])
+        op = ops.takes_operand(T, w["o"])
+        r = ops.gated_recurrence(self._gate_logits(ops, u), self.bs, w["ra.b"], w["ri.b"], w["lam"], self.decay, u, D[:, :n],
+                                 ctx.pool.state[:, at + self.conv_floats:at + self.conv_floats + n], ctx, operand=op)
+        return [(ops.operand_linear(r, w["o"]) if op else ops.linear(r, w["o"]), None, 1.0)]
+
+
+class TokenSide:
+    """What the token itself adds in every layer:  y = W_proj (gelu(W_gate x) * e), e the layer's slice of a table's row of
+    the token (`dim` numbers; the model binds `table`);  x += y / sqrt(mean(y^2) + eps) * norm."""
+
+    def __init__(self, index: int, dim: int, width: int):
+        self.index, self.dim, self.W = index, int(dim), width
+        self.table: Optional[torch.Tensor] = None       # (vocab, dim): columns of the model's table
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def manifest(self, p: str):
+        return [(p + "gate", (self.dim, self.W)), (p + "proj", (self.W, self.dim)), (p + "norm", (self.W,))]
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        return dict(self.manifest(p))
+
+    def pack(self, p: str, ck, view):
+        for n, _ in self.manifest(p):
+            view(n).copy_(ck[n])
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n[len(p):]: view(n) for n, _ in self.manifest(p)}
+
+    def on_tensor_cores(self, ops: LayerOps, T: int) -> bool:
+        return ops.takes_operand(T, self.w["gate"]) and ops.takes_operand(T, self.w["proj"])
+
+    def rows(self, ctx: StepCtx, x: torch.Tensor, pending: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """pending: rows that are still to be added to x (few rows: the gate's product reads the sum itself)"""
+        ops, w, T = ctx.ops, self.w, x.shape[0]
+        if pending is None and self.on_tensor_cores(ops, T):
+            z = ops.linear(x, w["gate"], operand=ctx.x_operand)
+            return ops.operand_linear(ops.table_gate_bf16(z, self.table, ctx.tokens), w["proj"])
+        z = ops.empty((T, self.dim))
+        ops.gemm(x, w["gate"], z, M=T, N_=self.dim, K=self.W, epi=EPI_TABLE_GATE, X2=pending, table=self.table, table_row=ctx.tokens)
+        return ops.linear(z, w["proj"])
+
+
+PRENORM_MIXERS = {"parallel": lambda i, c, w: PairedMixer(i, c, w, GroupedAttention(i, c["left"], w, qk_norm="unit", sink="unit", bias=True),
+                                                          MatrixMemory(i, c["right"], w)),
+                  "rglru": GatedRecurrence}
+PRENORM_FEEDFORWARDS = {"dense": GatedDense}
+
+
+class PreNormLayer:
+    """x <- x + mixer(N1(x));  x <- x + ff(N2(x));  x <- x + token input,  N(y) = y / sqrt(mean(y^2) + eps) * w; a layer may
+    have no feed-forward, a model no token input (`side_dim` 0).  The residual stream, its sums and all norms are fp32; the
+    residual update of a sublayer, the norms of its branches and the norm that the next sublayer reads are one launch, which in a
+    prompt also writes the bf16 operand rows of the next product."""
+
+    def __init__(self, index: int, cfg: dict, width: int, side_dim: int = 0):
+        self.index, self.W = index, width
+        if cfg["type"] not in PRENORM_MIXERS:
+            raise ValueError(f"layer {index}: unknown mixer type {cfg['type']!r} (have {sorted(PRENORM_MIXERS)})")
+        self.mixer = PRENORM_MIXERS[cfg["type"]](index, cfg["mixer"], width)
+        f = cfg.get("mlp")
+        if f is not None and f.get("kind") not in PRENORM_FEEDFORWARDS:
+            raise ValueError(f"layer {index}: unknown feed-forward kind {f.get('kind')!r} (have {sorted(PRENORM_FEEDFORWARDS)})")
+        self.ff = None if f is None else PRENORM_FEEDFORWARDS[f["kind"]](index, f, width)
+        self.side = TokenSide(index, side_dim, width) if side_dim else None
+        self.kv_dim, self.state_floats = self.mixer.kv_dim, self.mixer.state_floats
+        self.w: Dict[str, torch.Tensor] = {}
+
+    def _own(self):
+        return ["norm1"] + (["norm2"] if self.ff is not None else [])
+
+    def _blocks(self):
+        return [("mix.", self.mixer)] + ([("mlp.", self.ff)] if self.ff is not None else []) + \
+               ([("side.", self.side)] if self.side is not None else [])
+
+    def manifest(self, p: str):
+        out = [(p + n, (self.W,)) for n in self._own()]
+        for s, b in self._blocks():
+            out += b.manifest(p + s)
+        return out
+
+    def checkpoint_tensors(self, p: str) -> Dict[str, tuple]:
+        out = {p + n: (self.W,) for n in self._own()}
+        for s, b in self._blocks():
+            out.update(b.checkpoint_tensors(p + s))
+        return out
+
+    def pack(self, p: str, ck, view):
+        for n in self._own():
+            view(p + n).copy_(ck[p + n])
+        for s, b in self._blocks():
+            b.pack(p + s, ck, view)
+        self.bind(p, view)
+
+    def bind(self, p: str, view):
+        self.w = {n: view(p + n) for n in self._own()}
+        for s, b in self._blocks():
+            b.bind(p + s, view)
+
+    def forward(self, ctx: StepCtx, x: torch.Tensor, normed: Optional[torch.Tensor] = None,
+                next_norm: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+        """normed: N1(x) if the launch before already made it (its operand rows are ctx.x_operand); extra: rows added to x after
+        this layer; next_norm: the weight of the norm that follows — the result is then returned (its operand rows in
+        ctx.x_operand)"""
+        ops = ctx.ops
+        n = normed
+        if n is None:
+            n, ctx.x_operand = ops.close_rows(x, [], ctx.eps, norm=self.w["norm1"])
+        branches = self.mixer.forward(ctx, n)
+        if self.ff is not None:
+            n, ctx.x_operand = ops.close_rows(x, branches, ctx.eps, norm=self.w["norm2"])
+            branches = [(self.ff.rows(ctx, n), None, 1.0)]
+        if self.side is not None:
+            if len(branches) == 1 and branches[0][1:] == (None, 1.0) and not self.side.on_tensor_cores(ops, x.shape[0]):
+                branches.append((self.side.rows(ctx, x, pending=branches[0][0]), self.side.w["norm"], 1.0))
+            else:
+                _, ctx.x_operand = ops.close_rows(x, branches, ctx.eps)
+                branches = [(self.side.rows(ctx, x), self.side.w["norm"], 1.0)]
+        n, ctx.x_operand = ops.close_rows(x, branches, ctx.eps, extra=extra, norm=next_norm, operand=next_norm is not None)
+        return n
 
 
 def assign_cache_layers(layers: List) -> int:

@@ -15,13 +15,14 @@ import torch
 
 from .. import _native as N
 
-EPI_NONE, EPI_RELU2, EPI_SOFTCAP, EPI_ADD, EPI_SCALE, EPI_GELU = 0, 1, 2, 3, 4, 5
+EPI_NONE, EPI_RELU2, EPI_SOFTCAP, EPI_ADD, EPI_SCALE, EPI_GELU, EPI_TABLE_GATE = 0, 1, 2, 3, 4, 5, 6
 ACT_NONE, ACT_RELU2, ACT_GELU, ACT_TANH = 0, 1, 2, 3     # activation codes of `to_bf16` (gelu: the exact, erf form)
 GELU_TANH_ALPHA, GELU_TANH_CUBIC = 1.5957691216057308, 0.044715     # z sigmoid(alpha (z + cubic z^3)) = the tanh form of gelu
 WAVELENGTH = "wavelength"     # first entry of a frequency scaling by wavelength (a YaRN scaling is four numbers)
 SM_COUNT = 148
 TC_MIN_ROWS = 128     # from this many rows on, a product of the bf16 serving mode runs on the tcgen05 GEMM
 WT_F32 = 3            # gemm_wt output mode: fp32 rows
+LRU_PART = 64         # a sequence of more rows than this is walked in parts by the gated recurrence (32 parts at most)
 SKINNY_ROWS = 16      # up to this many rows a product runs on the warp-per-weight-row kernel
 
 
@@ -83,6 +84,54 @@ class LayerOps:
         self._ok(self.lib.b200_lm_embed(tokens.data_ptr(), table.data_ptr(), float(scale), x.data_ptr(), T, W, V,
                                         self.s), "lm_embed")
         return x
+
+    def embed_bigram(self, tokens: torch.Tensor, table: torch.Tensor, scale: float, bigram: torch.Tensor, mul_prev: int,
+                     mul_cur: int, state: torch.Tensor, ctx, keep: bool = False, norm: Optional[torch.Tensor] = None,
+                     eps: float = 0.0):
+        """-> (x, second copy or None, normed rows or None, their operand rows or None).  x[t] = table[token] * scale +
+        bigram[(previous token * mul_prev + token * mul_cur) mod buckets], buckets = the table's rows - 1; a sequence's first
+        token takes the last row.  state (slots, >= 1): the slot's number that holds the token before the step; norm: weight of
+        the RMS norm that follows (made in the same launch)"""
+        T, (V, W) = tokens.shape[0], table.shape
+        first, seqs, G = ctx.seq_tables()
+        x = self.empty((T, W))
+        kept = self.empty((T, W)) if keep else None
+        xn = self.empty((T, W)) if norm is not None else None
+        xb = self.empty((T, (W + 63) // 64 * 64), torch.bfloat16) if norm is not None and self.tc_ok(T, W) else None
+        self._ok(self.lib.b200_lm_embed_bigram(
+            tokens.data_ptr(), table.data_ptr(), float(scale), bigram.data_ptr(), bigram.shape[0] - 1, int(mul_prev), int(mul_cur),
+            state.data_ptr(), state.stride(0), ctx.slot.data_ptr(), ctx.pos.data_ptr(), first.data_ptr(), seqs.data_ptr(), G,
+            int(ctx.segments is None), x.data_ptr(), N.ptr(kept), N.ptr(norm), float(eps), N.ptr(xn), N.ptr(xb),
+            xb.stride(0) if xb is not None else 0, T, W, V, self.s), "lm_embed_bigram")
+        return x, kept, xn, xb
+
+    def close_rows(self, x: torch.Tensor, branches, eps: float, *, extra: Optional[torch.Tensor] = None,
+                   norm: Optional[torch.Tensor] = None, operand: bool = True):
+        """x (T, N) += sum of mult * N(y) over branches [(y, w, mult)] (w None: y itself) + extra; -> (N(x) with weight `norm`
+        or None, bf16 operand rows of it — without `norm`, of x — where the step's products run on the tensor cores)"""
+        T, n = x.shape
+        out = self.empty((T, n)) if norm is not None else None
+        xb = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16) if operand and self.tc_ok(T, n) else None
+        args = []
+        for i in range(3):
+            if i < len(branches):
+                y, w, m = branches[i]
+                args += [y.data_ptr(), y.stride(0), N.ptr(w), float(m)]
+            else:
+                args += [0, 0, 0, 0.0]
+        self._ok(self.lib.b200_lm_close_rows(
+            x.data_ptr(), x.stride(0), len(branches), *args, N.ptr(extra), extra.stride(0) if extra is not None else 0, N.ptr(norm),
+            float(eps), N.ptr(out), n, N.ptr(xb), xb.stride(0) if xb is not None else 0, T, n, self.s), "lm_close_rows")
+        return out, xb
+
+    def table_gate_bf16(self, z: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor) -> torch.Tensor:
+        """bf16 operand rows (T, ceil64(n)) of gelu(z) * table[token]; table (vocab, n): columns of a wider table"""
+        T, n = z.shape
+        out = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16)
+        self._ok(self.lib.b200_lm_table_gate_bf16(z.data_ptr(), z.stride(0), table.data_ptr(), table.stride(0), table.shape[0],
+                                                  tokens.data_ptr(), out.data_ptr(), n, out.stride(0), T, self.s),
+                 "lm_table_gate_bf16")
+        return out
 
     def inv_freq(self, base: float, dims: int, scaling: Optional[tuple] = None) -> torch.Tensor:
         """f_i = base^(-2i/dims), i < dims/2, computed in double precision on the host (once per rotation).
@@ -243,15 +292,19 @@ class LayerOps:
         return lists, count
 
     def gemm(self, X, W, Y, *, M, N_, K, ldx=None, xb=0, ldw=None, wb=0, ldy=None, yb=0, batch=1, bias=None,
-             lists=None, count=None, x_div=1, epi=EPI_NONE, epi_param=0.0, compact=0, exact_x: bool = False):
+             lists=None, count=None, x_div=1, epi=EPI_NONE, epi_param=0.0, compact=0, exact_x: bool = False,
+             X2: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, table_row: Optional[torch.Tensor] = None):
         """Y[b][r][:] = epi(X[b][r'] . W[b]^T + bias); strides in elements (default: the tensors' own rows).
         compact: an upper bound of the batches that have rows (a decode step: rows x top experts of many);
-        exact_x: the rows of X are not rounded to bf16 in the serving mode either (a router's input)"""
+        exact_x: the rows of X are not rounded to bf16 in the serving mode either (a router's input); X2: the rows
+        multiplied are X + X2; EPI_TABLE_GATE: gelu (tanh form) of the product times table[table_row[row]]"""
         self._ok(self.lib.b200_lm_gemm_rows(
             X.data_ptr(), X.stride(0) if ldx is None else ldx, xb, W.data_ptr(), K if ldw is None else ldw, wb,
             N.ptr(bias), Y.data_ptr(), Y.stride(0) if ldy is None else ldy, yb, N.ptr(lists),
             lists.stride(0) if lists is not None else 0, N.ptr(count), x_div, M, N_, K, batch, epi, float(epi_param),
-            int(not self.exact and not exact_x), int(M <= SKINNY_ROWS), int(compact), self.s), "lm_gemm_rows")
+            int(not self.exact and not exact_x), int(M <= SKINNY_ROWS), int(compact), N.ptr(X2),
+            X2.stride(0) if X2 is not None else 0, N.ptr(table), table.stride(0) if table is not None else 0, N.ptr(table_row),
+            table.shape[0] if table is not None else 0, self.s), "lm_gemm_rows")
 
     # ---- the tensor-core path of prompt steps (bf16 serving mode) ----------------------------------------
     def tc_ok(self, rows: int, *ks: int) -> bool:
@@ -294,8 +347,11 @@ class LayerOps:
         """fp32 rows -> (T, 2 ceil64(K)) bf16 = [hi | lo] with hi = bf16(x), lo = bf16(x - hi): sixteen more mantissa
         bits of x reach the tensor cores than with one rounded part (K a multiple of 4)"""
         T, Kp = X.shape[0], (K + 63) // 64 * 64
-        with torch.cuda.stream(self.stream):
-            out = torch.zeros((T, 2 * Kp), dtype=torch.bfloat16, device=self.device)
+        if Kp == K:
+            out = self.empty((T, 2 * Kp), torch.bfloat16)
+        else:
+            with torch.cuda.stream(self.stream):
+                out = torch.zeros((T, 2 * Kp), dtype=torch.bfloat16, device=self.device)
         self._ok(self.lib.b200_f32_split(X.data_ptr(), X.stride(0), out.data_ptr(), 2 * Kp, Kp, T, K, self.s), "f32_split")
         return out
 
@@ -324,10 +380,11 @@ class LayerOps:
                                                    N_, K, self.s), "gemm_wt_f32_grouped")
 
     def tc_gemm_heads(self, Xb: torch.Tensor, W: torch.Tensor, Y: torch.Tensor, *, H: int, N_: int, K: int,
-                      x_cols: int, x_group_cols: int, c_group_cols: int):
-        """Y[:, g * c_group_cols : + N_] = Xb[:, g * x_group_cols : + K] . W[g]^T for every head g, ONE tcgen05 launch"""
+                      x_cols: int, x_group_cols: int, c_group_cols: int, parts: int = 1):
+        """Y[:, g * c_group_cols : + N_] = Xb[:, g * x_group_cols : + K] . W[g]^T for every head g, ONE tcgen05 launch;
+        parts = 2: a head's columns are the [hi | lo] halves of K fp32 numbers"""
         self._ok(self.lib.b200_gemm_wt_f32_heads(Xb.data_ptr(), Xb.stride(0), x_cols, x_group_cols, W.data_ptr(), K,
-                                                 Y.data_ptr(), Y.stride(0), c_group_cols, Xb.shape[0], H, N_, K, self.s),
+                                                 Y.data_ptr(), Y.stride(0), c_group_cols, Xb.shape[0], H, N_, K, int(parts), self.s),
                  "gemm_wt_f32_heads")
 
     def rows_scatter(self, X: torch.Tensor, dst_map: torch.Tensor, out: torch.Tensor, rows: int):
@@ -372,6 +429,23 @@ class LayerOps:
         self.gemm(X, W, Y, M=T, N_=n, K=K, ldw=ldw, bias=bias, epi=EPI_ADD if add else epi, epi_param=epi_param,
                   exact_x=exact_x)
         return Y
+
+    def takes_operand(self, T: int, W: torch.Tensor) -> bool:
+        """a product of T rows with W runs on the tensor cores, so that the launch before it may write its bf16 operand rows"""
+        return self.tc_ok(T, W.shape[1], W.stride(0)) and W.data_ptr() % 16 == 0
+
+    def operand_linear(self, Xb: torch.Tensor, W: torch.Tensor) -> torch.Tensor:
+        """Y = X . W^T for rows that exist only as bf16 operand rows (T, ceil64(K))"""
+        n, K = W.shape
+        Y = self.empty((Xb.shape[0], n))
+        try:
+            self.tc_gemm(Xb, W, Y, N_=n, K=K, ldw=W.stride(0))
+            return Y
+        except N.B200Error as e:
+            self.tc_refused(e)
+        with torch.cuda.stream(self.stream):
+            X = Xb[:, :K].float()
+        return self.linear(X, W)
 
     # ---- sequences of a step, and the mixers that carry a state along them (csrc/mixer_ops.cu) -------------------
     def seq_tables(self, segments, T: int):
@@ -435,20 +509,20 @@ class LayerOps:
                  "lm_qkv_post")
 
     def head_qkv_post(self, Q, K, V, cache_layer, slot, pos, cs, H, G, dim, vdim, rot_dims, *, q_norm=None, k_norm=None,
-                      eps: float = 0.0, pairs: bool = False):
+                      eps: float = 0.0, pairs: bool = False, unit: bool = False):
         """`qkv_post` with everything per head: q_norm / k_norm (dim,): RMS norm of every head times ONE weight for all
-        heads; pairs: the rotation pairs (2i, 2i + 1).  V may be K itself"""
+        heads; unit: such norms without a weight; pairs: the rotation pairs (2i, 2i + 1).  V may be K itself"""
         self._ok(self.lib.b200_lm_head_qkv_post(
             Q.data_ptr(), Q.stride(0), K.data_ptr(), K.stride(0), V.data_ptr(), V.stride(0), cache_layer.data_ptr(),
             int(cache_layer.dtype == torch.bfloat16), cache_layer.stride(0), cache_layer.stride(1), slot.data_ptr(),
             pos.data_ptr(), cs.data_ptr(), H, G, dim, vdim, rot_dims, int(pairs), N.ptr(q_norm), N.ptr(k_norm), float(eps),
-            Q.shape[0], self.s), "lm_head_qkv_post")
+            int(unit), Q.shape[0], self.s), "lm_head_qkv_post")
 
     def sink_attention(self, Q, cache_layer, slot, pos, out, sink, H, G, dim, vdim, scale, chunk=0, window=0,
-                       n_split=None, bias_exp: float = 0.0, unit_sink: bool = False):
+                       n_split=None, bias_exp: float = 0.0, unit_sink: bool = False, softcap: float = 0.0):
         """n_split None: enough blocks per (token, kv head) to fill the GPU when the step has few tokens, 1 for prompts;
         bias_exp > 0: 2^(-bias_exp (h + 1) / H) times the distance to the key is taken off head h's scores; unit_sink:
-        the softmax's denominator also holds 1"""
+        the softmax's denominator also holds 1; softcap > 0: a score s becomes softcap tanh(s / softcap)"""
         T = Q.shape[0]
         if n_split is None:
             rep = H // G
@@ -461,7 +535,7 @@ class LayerOps:
             Q.data_ptr(), Q.stride(0), cache_layer.data_ptr(), int(cache_layer.dtype == torch.bfloat16),
             cache_layer.stride(0), cache_layer.stride(1), slot.data_ptr(), pos.data_ptr(), out.data_ptr(), out.stride(0),
             N.ptr(sink), H, G, dim, vdim, float(scale), int(chunk), int(window), float(bias_exp), int(unit_sink),
-            N.ptr(part), n_split, T, self.s),
+            float(softcap), N.ptr(part), n_split, T, self.s),
             "lm_sink_attention")
 
     def heads_to_bf16(self, q: torch.Tensor, rep: int, dim: int) -> torch.Tensor:
@@ -473,12 +547,12 @@ class LayerOps:
         return out
 
     def sink_softmax_bf16(self, S, pos, rep, sink, scale, chunk, window, key0, P, bias_exp: float = 0.0, head0: int = 0,
-                          H: int = 1, unit_sink: bool = False, split: bool = False):
+                          H: int = 1, unit_sink: bool = False, split: bool = False, softcap: float = 0.0):
         """head0, H: the first head of the rows' group and the number of heads (they fix the slopes of the distance bias);
         split: P (rows, 2 Sp) gets every probability as two bf16 parts [hi | lo], the operand of `tc_gemm(parts=2)`"""
         self._ok(self.lib.b200_lm_sink_softmax_bf16(S.data_ptr(), S.stride(0), pos.data_ptr(), rep, N.ptr(sink), float(scale),
                                                     int(chunk), int(window), int(key0), float(bias_exp), int(head0), int(H),
-                                                    int(unit_sink), int(split), P.data_ptr(), P.stride(0),
+                                                    int(unit_sink), int(split), float(softcap), P.data_ptr(), P.stride(0),
                                                     S.shape[0], P.shape[1] // 2 if split else P.shape[1], self.s),
                  "lm_sink_softmax_bf16")
 
@@ -525,6 +599,49 @@ class LayerOps:
             N.ptr(decay_logits), decay_logits.stride(0) if decay_logits is not None else 0, N.ptr(bonus),
             N.ptr(prep), int(part_len) if scratch is not None else 0, n_parts, N.ptr(scratch), max_rows, T, self.s),
             "lm_linear_state")
+
+    def gated_recurrence(self, G: torch.Tensor, bs: int, rb: torch.Tensor, ib: torch.Tensor, lam: torch.Tensor, c: float,
+                         u: torch.Tensor, y: torch.Tensor, state: torch.Tensor, ctx, operand: bool = False) -> torch.Tensor:
+        """log a = -c sigmoid(G_r + rb) softplus(lam), S <- a S + sqrt(1 - a^2) sigmoid(G_i + ib) u, -> S gelu(y); G (T, 2 n) in
+        blocks [r: bs | i: bs], overwritten; u, y (T, n); state (slots, n) fp32 view of the pool.  operand: the result as bf16
+        operand rows (T, ceil64(n)).  A long sequence is walked in parts at the same time"""
+        _, seqs, n_seq = ctx.seq_tables()
+        T, n = u.shape
+        longest = max(k for _, k, _, _ in ctx.segments) if ctx.segments else 1
+        part_len, n_parts, part = 0, 1, None
+        if longest > LRU_PART:
+            part_len = max(LRU_PART, -(-longest // 32))
+            n_parts = -(-longest // part_len)
+            part = self.empty((n_seq * n * (2 * n_parts + 1),))
+        out = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16) if operand else self.empty((T, n))
+        self._ok(self.lib.b200_lm_gated_recurrence(
+            G.data_ptr(), G.stride(0), int(bs), rb.data_ptr(), ib.data_ptr(), lam.data_ptr(), float(c), u.data_ptr(), u.stride(0),
+            y.data_ptr(), y.stride(0), state.data_ptr(), state.stride(0), seqs.data_ptr(), n_seq, ctx.slot.data_ptr(),
+            ctx.pos.data_ptr(), n, 0 if operand else out.data_ptr(), out.stride(0), out.data_ptr() if operand else 0,
+            out.stride(0) if operand else 0, part_len, n_parts, N.ptr(part), self.s), "lm_gated_recurrence")
+        return out
+
+    def matrix_memory(self, q, k, v, gi, gf, gate, w, state, ctx, *, H: int, dim: int, vdim: int, cap: float, q_scale: float,
+                      eps: float, operand: bool = False) -> torch.Tensor:
+        """the matrix memory with exponential gates (csrc/recurrent_ops.cu) up to its gated output (T, H vdim); gi, gf (T, H) the
+        gates' logits; state (slots, >= H (dim (vdim + 1) + 1)) fp32 view of the pool; operand: bf16 operand rows.  A step of more
+        than SKINNY_ROWS rows takes its sequences 64 tokens at a time"""
+        _, seqs, n_seq = ctx.seq_tables()
+        T = q.shape[0]
+        longest = max(n for _, n, _, _ in ctx.segments) if ctx.segments else 1
+        scratch, n_bytes = None, 0
+        if longest > SKINNY_ROWS:
+            n_bytes = self.lib.b200_lm_matrix_memory_scratch(T, n_seq, H, dim, vdim)
+            scratch = self.empty(((n_bytes + 15) // 16 * 4,))
+        n = H * vdim
+        out = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16) if operand else self.empty((T, n))
+        self._ok(self.lib.b200_lm_matrix_memory(
+            q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), gi.data_ptr(), gi.stride(0),
+            gf.data_ptr(), gf.stride(0), float(cap), float(q_scale), gate.data_ptr(), gate.stride(0), w.data_ptr(), float(eps),
+            state.data_ptr(), state.stride(0), seqs.data_ptr(), n_seq, ctx.slot.data_ptr(), ctx.pos.data_ptr(), H, dim, vdim,
+            0 if operand else out.data_ptr(), out.stride(0), out.data_ptr() if operand else 0, out.stride(0) if operand else 0,
+            N.ptr(scratch), n_bytes, longest, T, self.s), "lm_matrix_memory")
+        return out
 
     def head_post(self, o, out, *, dv, gate=None, gate_per_head=False, gate_silu=False, w=None, eps=0.0, span=0,
                   scale=1.0, gate_first=False):
