@@ -511,7 +511,7 @@ def c4_leg(dev, args):
 
 
 # ------------------------------------------------------------------------------------------------------------
-# `--design buzopel | sonulorn | lilosun | vadelix | futidra`: prefill and decode throughput of a decoder design assembled from decoder_blocks
+# `--design buzopel | sonulorn | lilosun | vadelix | futidra | nomivik`: prefill and decode throughput of a decoder design assembled from decoder_blocks
 # over the layer ops (Buzopel: latent attention + expert mixture; Sonulorn: sink attention, matrix-state mixers and a
 # clamped gated feed-forward behind one shared input projection; Lilosun: windowed gated latent attention and state-space
 # mixers in scaled pre-norm layers with a grouped expert mixture — also beside Buzopel, the closest design on the same
@@ -753,12 +753,58 @@ def _futidra_account(m, z, T):
     return act_w, other, mix_flops
 
 
+# Nomivik at the layer sizes of the designs above: windowed grouped attention beside a matrix memory with exponential gates,
+# gated linear recurrences of 5/4 of the width, silu-gated units, a token input of 256 numbers per layer.  Beside it Sonulorn
+# at equal width, depth, head sizes, feed-forward and window: the closest design on the same engine (attention beside a
+# matrix state, recurrent layers, gated dense units).
+NOMIVIK_SIZES = {
+    "2048w": dict(SONULORN_SIZES["2048w"], window=1024, lru=2560, blocks=10, side=256, buckets=65536),
+    "4096w": dict(SONULORN_SIZES["4096w"], window=1024, lru=5120, blocks=20, side=256, buckets=65536),
+}
+
+
+def _nomivik_config(z):
+    H, d = z["heads"], z["dim"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    left = {"heads": H, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "mask": {"size": z["window"]}, "scale": d ** -0.5,
+            "softcap": 50.0, "rot": {"base": 1000000.0, "dims": d // 2}}
+    pair = {"left": left, "right": {"heads": H, "dim": d, "vdim": d, "gate_cap": 15.0}}
+    lru = {"width": z["lru"], "blocks": z["blocks"], "conv": 4}
+    layers = [{"type": "parallel", "mixer": pair, "mlp": mlp}, {"type": "rglru", "mixer": lru, "mlp": mlp},
+              {"type": "parallel", "mixer": pair, "mlp": mlp}, {"type": "rglru", "mixer": lru, "mlp": mlp}]
+    return {"architecture": "Nomivik", "vocab": z["vocab"], "width": z["width"], "layers": layers[:z["layers"]],
+            "norm": {"eps": 1e-6}, "token_side": {"dim": z["side"]},
+            "embedding": {"bigram": {"buckets": z["buckets"], "mul_prev": 7919, "mul_cur": 31}}}
+
+
+def _nomivik_model(z, dev):
+    from mlx_vlm_b200.models.nomivik import Model as NModel, ModelConfig as NConfig
+    return NModel(NConfig.from_dict(_nomivik_config(z)), device=dev).init_random(0)
+
+
+def _nomivik_account(m, z, T):
+    from mlx_vlm_b200.models.decoder_blocks import PairedMixer
+    W = z["width"]
+    act_w, other, mix_flops = 0, 8 * m.state_floats, 0.0      # the fp32 state is read and written once per token
+    for run in m.runs:
+        L = m.layers[run.layer]
+        act_w += sum(t.numel() for t in L.mixer.w.values()) + (3 * L.ff.ff * W if L.ff is not None else 0) + 2 * L.side.dim * W
+        if isinstance(L.mixer, PairedMixer):
+            a, r = L.mixer.left, L.mixer.right
+            # visible keys of a query, averaged over the prompt; a decoded token after it reads a whole window
+            mean_seen = sum(min(p + 1, a.window or p + 1) for p in range(T)) / T
+            mix_flops += 2 * a.H * (a.dim + a.vdim) * mean_seen + 4 * r.H * r.dim * r.vdim
+            other += 2 * a.kv_dim * min(a.window or T, T)
+    return act_w, other, mix_flops
+
+
 # design -> (sizes, model factory, byte / flop accounting, closest design on the same engine measured beside it or None)
 DESIGNS = {"buzopel": (DESIGN_SIZES, _buzopel_model, _buzopel_account, None),
            "sonulorn": (SONULORN_SIZES, _sonulorn_model, _sonulorn_account, None),
            "lilosun": (LILOSUN_SIZES, _lilosun_model, _lilosun_account, ("buzopel_equal_size", _buzopel_model, _buzopel_account)),
            "vadelix": (VADELIX_SIZES, _vadelix_model, _vadelix_account, ("lilosun_equal_size", _lilosun_model, _lilosun_account)),
-           "futidra": (FUTIDRA_SIZES, _futidra_model, _futidra_account, ("sonulorn_equal_size", _sonulorn_model, _sonulorn_account))}
+           "futidra": (FUTIDRA_SIZES, _futidra_model, _futidra_account, ("sonulorn_equal_size", _sonulorn_model, _sonulorn_account)),
+           "nomivik": (NOMIVIK_SIZES, _nomivik_model, _nomivik_account, ("sonulorn_equal_size", _sonulorn_model, _sonulorn_account))}
 
 
 def _measure_layered(m, account, z, T, n_dec, rows, ids, args, timed, hbm, tpk):
@@ -889,7 +935,7 @@ def main():
     ap.add_argument("--no-mega", action="store_true")
     ap.add_argument("--mega-mode", type=int, default=None,
                     help="decode kernel: 0 per-phase kernels, 1 k_mega (CUDA cores), 2 k_mega_tc (tcgen05)")
-    ap.add_argument("--design", default=None, choices=["buzopel", "sonulorn", "lilosun", "vadelix", "futidra"],
+    ap.add_argument("--design", default=None, choices=["buzopel", "sonulorn", "lilosun", "vadelix", "futidra", "nomivik"],
                     help="instead of the default workload: prefill / decode throughput of this decoder design at "
                          "layer sizes of real models, beside the closest existing model at equal size")
     ap.add_argument("--design-sizes", default="", help="comma-separated subset of the sizes (default: all)")
