@@ -1391,6 +1391,54 @@ __global__ void sink_softmax_bf16_kernel(float* __restrict__ S, long lds, const 
   const float sk = sink ? bf2f(sink[r % rep]) : (unit_sink ? 0.f : -INFINITY);
   const float slope = bias_exp > 0.f ? exp2f(-bias_exp * (float)(head0 + (int)(r % rep) + 1) / (float)H) : 0.f;
   // the score of column j: scale s_j - slope (distance to the query); j1 - j is that distance
+  constexpr int PER = 8;
+  if (j1 - j0 < PER * (int)blockDim.x) {  // a row that fits the block's registers: every score is read once
+    float e[PER];
+    float m = sk;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int j = j0 + threadIdx.x + i * blockDim.x;
+      e[i] = j <= j1 ? s[j] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int j = j0 + threadIdx.x + i * blockDim.x;
+      if (j <= j1) {
+        float a = e[i] * scale;
+        if (softcap > 0.f) a = softcap * tanhf(a / softcap);
+        e[i] = a - slope * (float)(j1 - j);
+        m = fmaxf(m, e[i]);
+      }
+    }
+    m = warp_max(m);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
+    __syncthreads();
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) m = fmaxf(m, red[i]);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (j0 + (int)(threadIdx.x + i * blockDim.x) <= j1) { e[i] = expf(e[i] - m); sum += e[i]; }
+    const float inv = 1.0f / (block_sum_fixed(sum, red) + ((sink || unit_sink) ? expf(sk - m) : 0.f));
+    for (int j = threadIdx.x; j < j0; j += blockDim.x) {
+      P[r * ldp + j] = f2bf(0.f);
+      if (split) P[r * ldp + Sp + j] = f2bf(0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int j = j0 + threadIdx.x + i * blockDim.x;
+      if (j <= j1) {
+        const float pr = e[i] * inv;
+        const bf16 hi = f2bf(pr);
+        P[r * ldp + j] = hi;
+        if (split) P[r * ldp + Sp + j] = f2bf(pr - bf2f(hi));
+      }
+    }
+    for (int j = j1 + 1 + threadIdx.x; j < Sp; j += blockDim.x) {
+      P[r * ldp + j] = f2bf(0.f);
+      if (split) P[r * ldp + Sp + j] = f2bf(0.f);
+    }
+    return;
+  }
   const float mul = softcap > 0.f ? 1.f : scale;
   auto sc = [&](int j) { return s[j] * mul - slope * (float)(j1 - j); };
   float m = sk;

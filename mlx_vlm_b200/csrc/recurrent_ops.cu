@@ -297,22 +297,91 @@ __device__ __forceinline__ void tile_mma(const float (*A)[MC_LD], const float (*
       for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
   }
 }
-// tile[k][r] = row r, number k0 + k of rows laid out along k in memory (zeros outside); times scale[r]
-__device__ __forceinline__ void load_rows_t(float (*tile)[MC_LD], const float* x, long ld, int n_rows, int k0, int K, const float* scale,
-                                            float mul) {
-  for (int e = threadIdx.x; e < MC * MC_K; e += MC_THREADS) {
-    const int r = e / MC_K, k = e % MC_K;
-    tile[k][r] = (r < n_rows && k0 + k < K) ? x[(long)r * ld + k0 + k] * (scale ? scale[r] * mul : mul) : 0.f;
+// A tile's numbers travel from memory through registers: the next tile is requested while the current one is multiplied.
+// Along: tile[k][r] = number k0 + k of row r (rows laid out along k), times mul scale[r]; a thread takes eight numbers of one
+// row (a whole sector), neighbouring lanes neighbouring rows.  Across: tile[k][c] = number c0 + c of row k0 + k, times
+// scale[k0 + k]; a thread takes four numbers of two rows.  VEC: everything starts on 16-byte boundaries, sizes are multiples of 4
+constexpr int MC_REGS = 8;
+static_assert(MC * MC_K == MC_THREADS * MC_REGS, "");
+template <bool VEC>
+struct Along {
+  const float* x; long ld; int n_rows, K; const float* scale; float mul;
+  __device__ __forceinline__ void request(int k0, float (&v)[MC_REGS]) const {
+    const int r = threadIdx.x % MC, k = k0 + threadIdx.x / MC * MC_REGS;
+#pragma unroll
+    for (int j = 0; j < MC_REGS; j += 4) {
+      if constexpr (VEC) {
+        const float4 a = (r < n_rows && k + j < K) ? *reinterpret_cast<const float4*>(x + (long)r * ld + k + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[j] = a.x; v[j + 1] = a.y; v[j + 2] = a.z; v[j + 3] = a.w;
+      } else {
+#pragma unroll
+        for (int e = j; e < j + 4; ++e) v[e] = (r < n_rows && k + e < K) ? x[(long)r * ld + k + e] : 0.f;
+      }
+    }
+  }
+  __device__ __forceinline__ void store(float (*tile)[MC_LD], int, const float (&v)[MC_REGS]) const {
+    const int r = threadIdx.x % MC, k = threadIdx.x / MC * MC_REGS;
+    const float f = scale ? scale[r] * mul : mul;
+#pragma unroll
+    for (int j = 0; j < MC_REGS; ++j) tile[k + j][r] = v[j] * f;
+  }
+};
+template <bool VEC>
+struct Across {
+  const float* x; long ld; int K, c0, C; const float* scale;
+  __device__ __forceinline__ void request(int k0, float (&v)[MC_REGS]) const {
+    const int c = c0 + threadIdx.x % (MC / 4) * 4;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int k = k0 + h * (MC_K / 2) + threadIdx.x / (MC / 4);
+      if constexpr (VEC) {
+        const float4 a = (k < K && c < C) ? *reinterpret_cast<const float4*>(x + (long)k * ld + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[4 * h] = a.x; v[4 * h + 1] = a.y; v[4 * h + 2] = a.z; v[4 * h + 3] = a.w;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[4 * h + e] = (k < K && c + e < C) ? x[(long)k * ld + c + e] : 0.f;
+      }
+    }
+  }
+  __device__ __forceinline__ void store(float (*tile)[MC_LD], int k0, const float (&v)[MC_REGS]) const {
+    const int c = threadIdx.x % (MC / 4) * 4;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int k = h * (MC_K / 2) + threadIdx.x / (MC / 4);
+      const float f = scale ? (k0 + k < K ? scale[k0 + k] : 0.f) : 1.f;
+      *reinterpret_cast<float4*>(&tile[k][c]) = make_float4(v[4 * h] * f, v[4 * h + 1] * f, v[4 * h + 2] * f, v[4 * h + 3] * f);
+    }
+  }
+};
+// acc += A B over K numbers (staged: A is already in shared memory, [k][MC_LD])
+template <class SA, class SB>
+__device__ __forceinline__ void tile_product(MemTile& tile, const SA& sa, const SB& sb, int K, float (&acc)[4][4]) {
+  float va[MC_REGS], vb[MC_REGS];
+  sa.request(0, va);
+  sb.request(0, vb);
+  for (int k0 = 0; k0 < K; k0 += MC_K) {
+    __syncthreads();
+    sa.store(tile.a, k0, va);
+    sb.store(tile.b, k0, vb);
+    __syncthreads();
+    if (k0 + MC_K < K) { sa.request(k0 + MC_K, va); sb.request(k0 + MC_K, vb); }
+    tile_mma(tile.a, tile.b, min(MC_K, K - k0), acc);
   }
 }
-// tile[k][c] = row k0 + k, number c0 + c; times scale[k0 + k]
-__device__ __forceinline__ void load_rows(float (*tile)[MC_LD], const float* x, long ld, int k0, int K, int c0, int C, const float* scale) {
-  for (int e = threadIdx.x; e < MC_K * MC; e += MC_THREADS) {
-    const int k = e / MC, c = e % MC;
-    tile[k][c] = (k0 + k < K && c0 + c < C) ? x[(long)(k0 + k) * ld + c0 + c] * (scale ? scale[k0 + k] : 1.f) : 0.f;
+template <class SB>
+__device__ __forceinline__ void tile_product_staged(MemTile& tile, const float (*PA)[MC_LD], const SB& sb, int K, float (&acc)[4][4]) {
+  float vb[MC_REGS];
+  sb.request(0, vb);
+  for (int k0 = 0; k0 < K; k0 += MC_K) {
+    __syncthreads();
+    sb.store(tile.b, k0, vb);
+    __syncthreads();
+    if (k0 + MC_K < K) sb.request(k0 + MC_K, vb);
+    tile_mma(PA + k0, tile.b, min(MC_K, K - k0), acc);
   }
 }
 
+template <bool VEC>
 __global__ void __launch_bounds__(MC_THREADS) memory_chunk_kernel(MemP p) {
   __shared__ MemTile tile;
   __shared__ float ws[MC];
@@ -362,13 +431,7 @@ __global__ void __launch_bounds__(MC_THREADS) memory_chunk_kernel(MemP p) {
   for (int i0 = 0; i0 < d; i0 += MC)
     for (int c0 = 0; c0 < dv; c0 += MC) {
       float acc[4][4] = {};
-      for (int s0 = 0; s0 < nc; s0 += MC_K) {
-        __syncthreads();
-        load_rows(tile.a, k, p.ldk, s0, nc, i0, d, ws);
-        load_rows(tile.b, v, p.ldv, s0, nc, c0, dv, nullptr);
-        __syncthreads();
-        tile_mma(tile.a, tile.b, min(MC_K, nc - s0), acc);
-      }
+      tile_product(tile, Across<VEC>{k, p.ldk, nc, i0, d, ws}, Across<VEC>{v, p.ldv, nc, c0, dv, nullptr}, nc, acc);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -385,8 +448,10 @@ __global__ void __launch_bounds__(MC_THREADS) memory_chunk_kernel(MemP p) {
   }
 }
 
-// start states, chunk after chunk; a thread per number of the head's S and n.  Every thread follows the running maximum
+// start states, chunk after chunk; a thread per number of the head's S and n.  The running maximum of 32 chunks at a time, and
+// from it what a chunk keeps of the state and what it puts, by one warp
 __global__ void memory_chain_kernel(MemP p) {
+  __shared__ float keep[32], put[32];
   const int seq = blockIdx.x, h = blockIdx.y, d = p.dim, dv = p.vdim;
   const long e = (long)blockIdx.z * blockDim.x + threadIdx.x, num = (long)d * (dv + 1);
   const int first = p.seqs[2 * seq], n = (p.seqs[2 * seq + 1] + MC - 1) / MC;
@@ -397,32 +462,45 @@ __global__ void memory_chain_kernel(MemP p) {
   float S = (ok && p.pos[first] > 0) ? *mine : 0.f;
   float m = p.mstart[(long)seq * p.H + h];
   constexpr int B = 8;                // chunks whose numbers are loaded together
-  for (int c0 = 0; c0 < n; c0 += B) {
-    float add[B];
-    double F[B], M[B];
+  for (int g0 = 0; g0 < n; g0 += 32) {
+    __syncthreads();
+    if (threadIdx.x < 32) {
+      const int lane = threadIdx.x, c = g0 + lane;
+      const long ch = (ch0 + min(c, n - 1)) * p.H + h;
+      double F = c < n ? p.tot[2 * ch] : 0.0, M = c < n ? p.tot[2 * ch + 1] : -INFINITY;
+      const double F1 = F, M1 = M;    // the chunk's own
 #pragma unroll
-    for (int j = 0; j < B; ++j) {
-      const long ch = (ch0 + min(c0 + j, n - 1)) * p.H + h;
-      add[j] = ok ? p.chunk[ch * num + e] : 0.f;
-      F[j] = p.tot[2 * ch];
-      M[j] = p.tot[2 * ch + 1];
-    }
-#pragma unroll
-    for (int j = 0; j < B; ++j)
-      if (c0 + j < n) {
-        const long ch = (ch0 + c0 + j) * p.H + h;
-        const float mn = (float)fmax(F[j] + (double)m, M[j]);
-        const float keep = expf((float)(F[j] + (double)m - (double)mn)), put = expf((float)(M[j] - (double)mn));
-        if (e == 0) p.m0[ch] = m;
-        if (ok) p.chunk[ch * num + e] = S;
-        S = fmaf(keep, S, put * add[j]);
-        m = mn;
+      for (int o = 1; o < 32; o <<= 1) {
+        const double fp = __shfl_up_sync(0xffffffffu, F, o), mp = __shfl_up_sync(0xffffffffu, M, o);
+        if (lane >= o) { M = fmax(mp + F, M); F += fp; }
       }
+      const float after = (float)fmax(F + (double)m, M);
+      float before = __shfl_up_sync(0xffffffffu, after, 1);
+      if (lane == 0) before = m;
+      keep[lane] = expf((float)(F1 + (double)before - (double)after));
+      put[lane] = expf((float)(M1 - (double)after));
+      if (c < n && blockIdx.z == 0) p.m0[ch] = before;
+      m = __shfl_sync(0xffffffffu, after, 31);       // (chunks past the end change nothing)
+    }
+    __syncthreads();
+    const int g1 = min(n, g0 + 32);
+    for (int c0 = g0; c0 < g1; c0 += B) {
+      float add[B];
+#pragma unroll
+      for (int j = 0; j < B; ++j) add[j] = ok ? p.chunk[((ch0 + min(c0 + j, n - 1)) * p.H + h) * num + e] : 0.f;
+#pragma unroll
+      for (int j = 0; j < B; ++j)
+        if (c0 + j < g1) {
+          if (ok) p.chunk[((ch0 + c0 + j) * p.H + h) * num + e] = S;
+          S = fmaf(keep[c0 + j - g0], S, put[c0 + j - g0] * add[j]);
+        }
+    }
   }
   if (ok) *mine = S;
   if (e == 0) st[(long)p.H * d * (dv + 1) + h] = m;
 }
 
+template <bool VEC>
 __global__ void __launch_bounds__(MC_THREADS) memory_out_kernel(MemP p) {
   extern __shared__ __align__(16) float sm[];
   MemTile& tile = *reinterpret_cast<MemTile*>(sm);
@@ -451,13 +529,7 @@ __global__ void __launch_bounds__(MC_THREADS) memory_out_kernel(MemP p) {
   }
   {
     float acc[4][4] = {};
-    for (int k0 = 0; k0 < d; k0 += MC_K) {
-      __syncthreads();
-      load_rows_t(tile.a, k, p.ldk, nc, k0, d, nullptr, 1.f);
-      load_rows_t(tile.b, q, p.ldq, nc, k0, d, nullptr, p.q_scale);
-      __syncthreads();
-      tile_mma(tile.a, tile.b, min(MC_K, d - k0), acc);
-    }
+    tile_product(tile, Along<VEC>{k, p.ldk, nc, d, nullptr, 1.f}, Along<VEC>{q, p.ldq, nc, d, nullptr, p.q_scale}, d, acc);
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -475,19 +547,8 @@ __global__ void __launch_bounds__(MC_THREADS) memory_out_kernel(MemP p) {
   }
   for (int c0 = 0; c0 < dv; c0 += MC) {
     float acc[4][4] = {};
-    for (int s0 = 0; s0 < nc; s0 += MC_K) {
-      __syncthreads();
-      load_rows(tile.b, v, p.ldv, s0, nc, c0, dv, nullptr);
-      __syncthreads();
-      tile_mma(P + s0, tile.b, min(MC_K, nc - s0), acc);
-    }
-    for (int k0 = 0; k0 < d; k0 += MC_K) {
-      __syncthreads();
-      load_rows_t(tile.a, q, p.ldq, nc, k0, d, ws, p.q_scale);
-      load_rows(tile.b, S, dv, k0, d, c0, dv, nullptr);
-      __syncthreads();
-      tile_mma(tile.a, tile.b, min(MC_K, d - k0), acc);
-    }
+    tile_product_staged(tile, P, Across<VEC>{v, p.ldv, nc, c0, dv, nullptr}, nc, acc);
+    tile_product(tile, Along<VEC>{q, p.ldq, nc, d, ws, p.q_scale}, Across<VEC>{S, dv, d, c0, dv, nullptr}, d, acc);
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -577,21 +638,26 @@ int b200_lm_matrix_memory(const float* q, long ldq, const float* k, long ldk, co
   const long chunks = (long)T / MC + n_seq + 1;
   p.F = (double*)scratch;
   p.tot = p.F + (long)T * H;
-  p.chunk = (float*)(p.tot + chunks * H * 2);
+  p.chunk = (float*)(p.F + ((long)T * H + chunks * H * 2 + 1) / 2 * 2);     // 16-byte aligned
   p.li = p.chunk + chunks * H * ((long)dim * (vdim + 1));
   p.ml = p.li + (long)T * H;
   p.m0 = p.ml + (long)T * H;
   p.mstart = p.m0 + chunks * H;
   const size_t smem = sizeof(MemTile) + (size_t)MC * MC_LD * 4 + (size_t)MC * vdim * 4;
   B200_REQUIRE(smem <= 200 * 1024, "lm_matrix_memory: values of %d numbers do not fit shared memory", vdim);
-  if (first_use_on_device(&g_mem_attr))
-    B200_CUDA(cudaFuncSetAttribute(memory_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  if (first_use_on_device(&g_mem_attr)) {
+    B200_CUDA(cudaFuncSetAttribute(memory_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(memory_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  }
+  const bool vec = ((dim | vdim | ldq | ldk | ldv) & 3) == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)p.chunk) & 15) == 0;
   const dim3 grid(cdiv(max_rows, MC), H, n_seq);
-  memory_chunk_kernel<<<grid, MC_THREADS, 0, cs>>>(p);
+  if (vec) memory_chunk_kernel<true><<<grid, MC_THREADS, 0, cs>>>(p);
+  else memory_chunk_kernel<false><<<grid, MC_THREADS, 0, cs>>>(p);
   B200_CHECK_LAUNCH();
   memory_chain_kernel<<<dim3(n_seq, H, cdiv((long)dim * (vdim + 1), 256)), 256, 0, cs>>>(p);
   B200_CHECK_LAUNCH();
-  memory_out_kernel<<<grid, MC_THREADS, smem, cs>>>(p);
+  if (vec) memory_out_kernel<true><<<grid, MC_THREADS, smem, cs>>>(p);
+  else memory_out_kernel<false><<<grid, MC_THREADS, smem, cs>>>(p);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }

@@ -69,6 +69,7 @@ so a prompt, a portion of a prompt, a decoded token and a batch of unequal reque
 """
 from __future__ import annotations
 
+from contextlib import nullcontext
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
@@ -1774,7 +1775,8 @@ class MatrixMemory:
 class PairedMixer:
     """An attention (`left`) and a matrix memory (`right`) that read the same input: half the sum of their outputs, each first
     RMS-normed over the width with a weight of its own (`left.out`, `right.out`).  All their input projections are ONE product,
-    the norms, the factors and the sum belong to the residual update."""
+    the norms, the factors and the sum belong to the residual update; the right one runs on a
+    second stream beside the left one."""
 
     def __init__(self, index: int, cfg: dict, width: int, left, right, factor: float = 0.5):
         self.index, self.W, self.left, self.right, self.factor = index, width, left, right, float(factor)
@@ -1825,10 +1827,17 @@ class PairedMixer:
         ops, w, T = ctx.ops, self.w, h.shape[0]
         D = ops.linear(h, w["in"], bias=w["in.b"], operand=ctx.x_operand)
         a, b = self.left.n_in, self.right.n_in
-        yl = ops.linear(self.left.attend(ctx, D[:, :a]), w["left.o"])
-        op = ops.takes_operand(T, w["right.o"])
-        r = self.right.mix(ctx, D[:, a:a + b], operand=op)
-        yr = ops.operand_linear(r, w["right.o"]) if op else ops.linear(r, w["right.o"])
+        ctx.seq_tables()                      # (made on the engine's stream)
+        # the two mixers do not wait for one another.  The first step of a size keeps to one stream: its products choose their
+        # tiles by timing them
+        with ops.beside() if ops.seen(("pair", self.index, (T + 63) // 64)) else nullcontext():
+            op = ops.takes_operand(T, w["right.o"])
+            r = self.right.mix(ctx, D[:, a:a + b], operand=op)
+            yr = ops.operand_linear(r, w["right.o"]) if op else ops.linear(r, w["right.o"])
+        try:
+            yl = ops.linear(self.left.attend(ctx, D[:, :a]), w["left.o"])
+        finally:
+            ops.join()
         return [(yl, w["left.out"], self.factor), (yr, w["right.out"], self.factor)]
 
 

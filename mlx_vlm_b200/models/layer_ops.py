@@ -22,7 +22,7 @@ WAVELENGTH = "wavelength"     # first entry of a frequency scaling by wavelength
 SM_COUNT = 148
 TC_MIN_ROWS = 128     # from this many rows on, a product of the bf16 serving mode runs on the tcgen05 GEMM
 WT_F32 = 3            # gemm_wt output mode: fp32 rows
-LRU_PART = 64         # a sequence of more rows than this is walked in parts by the gated recurrence (32 parts at most)
+LRU_PART = 32         # a sequence of more rows than this is walked in parts by the gated recurrence (64 parts at most)
 SKINNY_ROWS = 16      # up to this many rows a product runs on the warp-per-weight-row kernel
 
 
@@ -37,6 +37,8 @@ class LayerOps:
         self._unit_seqs = {}
         self._on_stream = False
         self.tc_enabled = True
+        self._seen = set()
+        self._side = self._join = None      # second stream, and the event at the end of what it was given
 
     @property
     def s(self) -> int:
@@ -71,6 +73,45 @@ class LayerOps:
                 return self.inner.__exit__(*exc)
 
         return _Ctx()
+
+    def beside(self):
+        """context: what is enqueued inside runs on a second stream, beside what the engine's stream gets from here to `join()`.
+        The second stream starts behind everything enqueued so far, and buffers made inside are its own: they may be read after
+        `join()`, and are free for the next such context, which starts behind their readers"""
+        ops = self
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.device)
+        main, side = self.stream, self._side
+
+        class _Ctx:
+            def __enter__(self):
+                fork = torch.cuda.Event()
+                fork.record(main)
+                side.wait_event(fork)
+                ops.stream = side
+                self.inner = torch.cuda.stream(side)
+                self.inner.__enter__()
+
+            def __exit__(self, *exc):
+                ops.stream = main
+                ops._join = torch.cuda.Event()
+                ops._join.record(side)
+                return self.inner.__exit__(*exc)
+
+        return _Ctx()
+
+    def seen(self, key) -> bool:
+        """whether this was asked before with the same key"""
+        if key in self._seen:
+            return True
+        self._seen.add(key)
+        return False
+
+    def join(self):
+        """the engine's stream goes on behind everything that `beside()` enqueued"""
+        if self._join is not None:
+            self.stream.wait_event(self._join)
+            self._join = None
 
     def to_device(self, arr, dtype=np.int32) -> torch.Tensor:
         t = torch.from_numpy(np.ascontiguousarray(arr, dtype=dtype)).pin_memory()
@@ -610,7 +651,7 @@ class LayerOps:
         longest = max(k for _, k, _, _ in ctx.segments) if ctx.segments else 1
         part_len, n_parts, part = 0, 1, None
         if longest > LRU_PART:
-            part_len = max(LRU_PART, -(-longest // 32))
+            part_len = max(LRU_PART, -(-longest // 64))
             n_parts = -(-longest // part_len)
             part = self.empty((n_seq * n * (2 * n_parts + 1),))
         out = self.empty((T, (n + 63) // 64 * 64), torch.bfloat16) if operand else self.empty((T, n))
