@@ -327,9 +327,11 @@ int b200_gemm_wt_f32_grouped(const void* X, long ldx, const void* W, long ldw, f
                              const int* tile_group, int n_tiles, int n_groups, int N, int K_w, void* stream);
 /* the per-head projections of one token set in ONE launch: head g multiplies columns [g * x_group_cols, + K_w) of
  * X [T, x_cols] (bf16; K_w % 64 == 0) by W[g] [N, K_w] and writes columns [g * c_group_cols, + N) of C32; n_parts = 2: the
- * columns of a head are the [hi | lo] halves of K_w fp32 numbers, both multiplied by W[g] */
+ * columns of a head are the [hi | lo] halves of K_w fp32 numbers, both multiplied by W[g]; w_group_cols > 0: W[g] is columns
+ * [g * w_group_cols, + K_w) of ONE [N, ..] matrix, X's groups are ceil64(K_w) columns, zero beyond K_w */
 int b200_gemm_wt_f32_heads(const void* X, long ldx, int x_cols, int x_group_cols, const void* W, long ldw, float* C32,
-                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, int n_parts, void* stream);
+                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, int n_parts, int w_group_cols,
+                           void* stream);
 
 /* ------------------------------------------------------------------------- */
 /* Lock-step batched decode (continuous batching; generate/ar.py:929-1390        */
@@ -543,14 +545,17 @@ int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, con
                          const float* b, long ldb, int delta, int dt_in, const void* skip, const float* wraw, long ldwr,
                          const void* bonus, float* prep, int part_len, int n_parts, float* part_scratch, int max_rows, int T,
                          void* stream);
-/* operands of the tensor-core attention of a prompt step: out[(t, r)] = bf16 of q[t][r * dim .. + dim) padded to Kp;
+/* operands of the tensor-core attention of a prompt step: out[(t, r)][g Kp ..] = bf16 of q[t][(g rep + r) dim .. + dim), padded to Kp;
  * P[(t, r)][j] = softmax over the visible keys key0 + j (and sink[r]) of scale * S[(t, r)][j], bf16, zero elsewhere;
  * split: P rows are [hi | lo] (Sp columns each), lo the rounding error of hi (the operand of a two-part product);
- * softcap > 0: scores become softcap tanh(scale S / softcap), which S then holds */
-int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int dim, void* out, int Kp, int T, void* stream);
+ * softcap > 0: scores become softcap tanh(scale S / softcap), which S may then hold; G > 1: the rows of G groups of `rep` heads
+ * side by side, S s_group and P p_group columns apart (sink and head0 are the first group's) */
+int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int G, int dim, void* out, int Kp, int T, void* stream);
+/* out[t][(g rep + r) dv + c] = x[t rep + r][g ldg + c]: heads computed side by side per key/value head, in head order */
+int b200_lm_regroup_heads(const float* x, long ldx, int ldg, int rep, int G, int dv, float* out, long ldo, int T, void* stream);
 int b200_lm_sink_softmax_bf16(float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
                               int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, float softcap,
-                              void* P, long ldp, int rows, int Sp, void* stream);
+                              void* P, long ldp, int G, long s_group, long p_group, int rows, int Sp, void* stream);
 /* out[t][c] = scale * o[t][c] * [rsqrt(mean over c's group of `span` + eps)] * [w[c mod w_len]] * [act(gate)];
  * gate_first: the gate is applied before the norm (the mean square is that of the gated numbers) */
 int b200_lm_head_post(const float* o, long ldi, const float* gate, long ldg, const void* w, int w_len, float eps, int span,

@@ -133,7 +133,7 @@ LM_SIGNATURES = {
     "b200_lm_argmax_rows": (_I, [_P, _L, _I, _P, _P, _I, _P]),
     "b200_lm_rows_to_bf16": (_I, [_P, _L, _P, _I, _P, _L, _I, _I, _I, _I, _P]),
     "b200_gemm_wt_f32_grouped": (_I, [_P, _L, _P, _L, _P, _L, _P, _I, _I, _I, _I, _P]),
-    "b200_gemm_wt_f32_heads": (_I, [_P, _L, _I, _I, _P, _L, _P, _L, _L, _I, _I, _I, _I, _I, _P]),
+    "b200_gemm_wt_f32_heads": (_I, [_P, _L, _I, _I, _P, _L, _P, _L, _L, _I, _I, _I, _I, _I, _I, _P]),
     "b200_lm_moe_tiles": (_I, [_P, _L, _P, _I, _I, _P, _I, _P, _P]),
     "b200_lm_moe_order": (_I, [_P, _L, _P, _I, _P, _P]),
     "b200_lm_rows_scatter": (_I, [_P, _L, _P, _P, _L, _I, _I, _P]),
@@ -152,8 +152,10 @@ LM_SIGNATURES = {
                                     _P]),
     "b200_lm_linear_state": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F,
                                   _P, _P, _L, _P, _P, _P, _L, _I, _I, _P, _P, _L, _P, _P, _I, _I, _P, _I, _I, _P]),
-    "b200_lm_heads_to_bf16": (_I, [_P, _L, _I, _I, _P, _I, _I, _P]),
-    "b200_lm_sink_softmax_bf16": (_I, [_P, _L, _P, _I, _P, _F, _I, _I, _I, _F, _I, _I, _I, _I, _F, _P, _L, _I, _I, _P]),
+    "b200_lm_heads_to_bf16": (_I, [_P, _L, _I, _I, _I, _P, _I, _I, _P]),
+    "b200_lm_regroup_heads": (_I, [_P, _L, _I, _I, _I, _I, _P, _L, _I, _P]),
+    "b200_lm_sink_softmax_bf16": (_I, [_P, _L, _P, _I, _P, _F, _I, _I, _I, _F, _I, _I, _I, _I, _F, _P, _L, _I, _L, _L, _I, _I,
+                                      _P]),
     "b200_lm_head_post": (_I, [_P, _L, _P, _L, _P, _I, _F, _I, _I, _I, _I, _I, _F, _P, _L, _I, _I, _P]),
     "b200_lm_glu_clamp": (_I, [_P, _L, _P, _L, _F, _F, _F, _F, _I, _P, _L, _I, _I, _P]),
     "b200_lm_glu_clamp_bf16": (_I, [_P, _L, _P, _L, _F, _F, _F, _F, _I, _P, _I, _I, _P, _I, _P]),

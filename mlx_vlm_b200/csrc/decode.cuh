@@ -199,7 +199,8 @@ struct WtExt {
   // column groups (the heads of a per-head projection over the SAME tokens): group g multiplies columns
   // [g * x_group_cols, + K) of X by the weight rows of group g and writes columns [g * c_group_cols, + N) of C32;
   // W holds col_groups x N rows, X has x_cols columns in all.  One launch, grid.y = col_groups x token tiles.
-  int col_groups = 0;
+  // w_group_cols > 0: the groups' weights are instead column ranges of the same N rows, that many columns apart.
+  int col_groups = 0, w_group_cols = 0;
   int x_group_cols = 0, x_cols = 0;
   long c_group_cols = 0;
 };

@@ -68,6 +68,7 @@ struct WtParams {
   const int* tile_group;  // grouped products: token tile y multiplies the weight rows of group tile_group[y] (< 0: empty)
   int col_groups, x_group_cols;  // column groups: blockIdx.y = group x token tile; X columns / C32 columns move with the group
   long c_group_cols;
+  int w_group_cols;  // > 0: the groups' weights are column ranges of the SAME rows, this many columns apart (else rows g N .. of W)
 };
 
 __device__ __forceinline__ uint32_t w_smem_u32(const void* p) {
@@ -195,7 +196,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
   const int rb = blockIdx.x;
   const int n0 = rb * (swiglu ? 64 : WT_ROWS);  // first output feature (SwiGLU: channel) of the tile
   int n0w = n0;                                 // first weight row of the tile (grouped: inside the tile's group)
-  int ty = blockIdx.y, xk0 = 0;                 // token tile; first X column (column groups)
+  int ty = blockIdx.y, xk0 = 0, wk0 = 0;        // token tile; first X and W column (column groups)
   long cg = 0;                                  // first C32 column (column groups)
   if (p.tile_group) {
     const int g = p.tile_group[blockIdx.y];
@@ -204,7 +205,8 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
   } else if (p.col_groups > 0) {
     const int tpg = gridDim.y / p.col_groups, g = ty / tpg;
     ty -= g * tpg;
-    n0w += g * p.N;
+    if (p.w_group_cols > 0) wk0 = g * p.w_group_cols;
+    else n0w += g * p.N;
     xk0 = g * p.x_group_cols;
     cg = (long)g * p.c_group_cols;
   }
@@ -233,7 +235,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
     for (int j = 0; j < cnt; ++j) {
       int kbw = kb0 + it * p.KS + j;
       if (p.kb_w > 0) kbw %= p.kb_w;
-      const int kc = kbw * WT_BK;
+      const int kc = kbw * WT_BK + wk0;
       if (swiglu) {
         w_tma_2d(sW + j * WT_WBLK, &tmW, &full_bar[s], kc, n0);
         w_tma_2d(sW + j * WT_WBLK + 64 * 128, &tmW, &full_bar[s], kc, p.inter + n0);
@@ -808,11 +810,15 @@ int gemm_wt(const void* X, long ldx, const void* W, const void* bias, const void
     if (ext->kb_w > 0) k_w = ext->k_w;
     p.tile_group = ext->tile_group;
     p.col_groups = ext->col_groups; p.x_group_cols = ext->x_group_cols; p.c_group_cols = ext->c_group_cols;
+    p.w_group_cols = ext->w_group_cols;
   }
   const bool heads = ext && ext->col_groups > 0;
   B200_REQUIRE(!heads || (mode == B200_WT_F32 && cfg.split == 1 && !bias && !ext->res32 && !ext->tile_group &&
                           ext->x_group_cols % 8 == 0 && ext->x_cols >= (ext->col_groups - 1) * ext->x_group_cols + k_w),
                "gemm_wt: column groups are fp32-output, unsplit, without bias / residual, 16-byte column offsets");
+  const bool w_cols = heads && ext->w_group_cols > 0;
+  B200_REQUIRE(!w_cols || (ext->w_group_cols % 8 == 0 && ext->ldw >= (long)(ext->col_groups - 1) * ext->w_group_cols + k_w),
+               "gemm_wt: weight columns of the groups need 16-byte offsets inside the rows");
   const bool grouped = ext && ext->tile_group;
   B200_REQUIRE(!grouped || (mode == B200_WT_F32 && ext->n_groups > 0 && cfg.split == 1 && !bias),
                "gemm_wt: grouped products are fp32-output, unsplit, without bias");
@@ -822,7 +828,8 @@ int gemm_wt(const void* X, long ldx, const void* W, const void* bias, const void
   B200_REQUIRE((size_t)cfg.stages * stage >= (size_t)WT_EPI_TOK * WT_ROWS * 4, "gemm_wt: ring smaller than the epilogue staging tile");
   CUtensorMap tw, tx;
   int rc = wt_tmap(W, (long)(ext && ext->ldw > 0 ? ext->ldw : k_w),
-                   grouped ? ext->n_groups * N : (heads ? ext->col_groups * N : N), k_w,
+                   grouped ? ext->n_groups * N : (heads && !w_cols ? ext->col_groups * N : N),
+                   w_cols ? (ext->col_groups - 1) * ext->w_group_cols + k_w : k_w,
                    mode == B200_WT_SWIGLU ? 64 : WT_ROWS, &tw);
   if (rc) return rc;
   if ((rc = wt_tmap(X, ldx, T, heads ? ext->x_cols : K, cfg.TN, &tx))) return rc;

@@ -1370,18 +1370,35 @@ __global__ void glu_clamp_bf16x4_kernel(const float* __restrict__ G, long ldg, c
 // zeros to Kp columns; and the softmax of their score rows against the keys at positions key0 .. key0 + n_keys - 1 —
 // visible: max(start of pos's block, pos - window + 1, key0) .. pos — with the sink logit of the row's head in the
 // denominator, written as bf16 probabilities (normalised in fp32 before the rounding), zero where nothing is seen
-__global__ void heads_to_bf16_kernel(const float* __restrict__ q, long ldq, int rep, int dim, bf16* __restrict__ out,
+__global__ void heads_to_bf16_kernel(const float* __restrict__ q, long ldq, int rep, int G, int dim, bf16* __restrict__ out,
                                      int Kp) {
   const int i = blockIdx.x, t = i / rep, r = i % rep;
-  const float* x = q + (long)t * ldq + r * dim;
-  for (int k = threadIdx.x; k < Kp; k += blockDim.x) out[(long)i * Kp + k] = f2bf(k < dim ? x[k] : 0.f);
+  const float* x = q + (long)t * ldq + (long)r * dim;
+  for (int e = threadIdx.x; e < G * Kp; e += blockDim.x) {
+    const int g = e / Kp, k = e - g * Kp;
+    out[(long)i * G * Kp + e] = f2bf(k < dim ? x[(long)g * rep * dim + k] : 0.f);
+  }
+}
+// the outputs of heads that were computed side by side per key/value head, in head order:
+// out[t][(g rep + r) dv + c] = x[t rep + r][g ldg + c]
+__global__ void regroup_heads_kernel(const float* __restrict__ x, long ldx, int ldg, int rep, int G, int dv, float* __restrict__ out,
+                                     long ldo) {
+  const long t = blockIdx.x;
+  for (int e = threadIdx.x; e < G * rep * dv; e += blockDim.x) {
+    const int h = e / dv, c = e - h * dv, g = h / rep, r = h - g * rep;
+    out[t * ldo + e] = x[(t * rep + r) * ldx + (long)g * ldg + c];
+  }
 }
 __global__ void sink_softmax_bf16_kernel(float* __restrict__ S, long lds, const int* __restrict__ pos, int rep,
                                          const bf16* __restrict__ sink, float scale, int chunk, int window, int key0,
                                          float bias_exp, int head0, int H, int unit_sink, int split, float softcap,
-                                         bf16* __restrict__ P, long ldp, int Sp) {
+                                         bf16* __restrict__ P, long ldp, long s_group, long p_group, int Sp) {
   __shared__ float red[32];
   const long r = blockIdx.x;
+  S += blockIdx.y * s_group;           // one of several groups of heads side by side
+  P += blockIdx.y * p_group;
+  head0 += blockIdx.y * rep;
+  if (sink) sink += blockIdx.y * rep;
   const int ps = pos[r / rep];
   int lo = key0;
   if (chunk > 0) lo = max(lo, (ps / chunk) * chunk);
@@ -1391,19 +1408,27 @@ __global__ void sink_softmax_bf16_kernel(float* __restrict__ S, long lds, const 
   const float sk = sink ? bf2f(sink[r % rep]) : (unit_sink ? 0.f : -INFINITY);
   const float slope = bias_exp > 0.f ? exp2f(-bias_exp * (float)(head0 + (int)(r % rep) + 1) / (float)H) : 0.f;
   // the score of column j: scale s_j - slope (distance to the query); j1 - j is that distance
-  constexpr int PER = 8;
-  if (j1 - j0 < PER * (int)blockDim.x) {  // a row that fits the block's registers: every score is read once
-    float e[PER];
+  constexpr int PER = 4;               // pairs of neighbouring columns per thread
+  const int b0 = j0 & ~1;
+  if (j1 - b0 < 2 * PER * (int)blockDim.x) {  // a row that fits the block's registers: every score is read once
+    const bool v2 = (lds & 1) == 0 && ((uintptr_t)S & 7) == 0, w2 = (ldp & 1) == 0 && (Sp & 1) == 0 && ((uintptr_t)P & 3) == 0;
+    float e[2 * PER];
     float m = sk;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      const int j = j0 + threadIdx.x + i * blockDim.x;
-      e[i] = j <= j1 ? s[j] : 0.f;
+      const int j = b0 + 2 * (threadIdx.x + i * blockDim.x);
+      if (v2 && j < j1) {                  // (columns j and j + 1 are both of the row)
+        const float2 a = *reinterpret_cast<const float2*>(s + j);
+        e[2 * i] = a.x; e[2 * i + 1] = a.y;
+      } else {
+        e[2 * i] = j <= j1 ? s[j] : 0.f;
+        e[2 * i + 1] = j + 1 <= j1 ? s[j + 1] : 0.f;
+      }
     }
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-      const int j = j0 + threadIdx.x + i * blockDim.x;
-      if (j <= j1) {
+    for (int i = 0; i < 2 * PER; ++i) {
+      const int j = b0 + 2 * (threadIdx.x + i / 2 * blockDim.x) + (i & 1);
+      if (j >= j0 && j <= j1) {
         float a = e[i] * scale;
         if (softcap > 0.f) a = softcap * tanhf(a / softcap);
         e[i] = a - slope * (float)(j1 - j);
@@ -1416,27 +1441,37 @@ __global__ void sink_softmax_bf16_kernel(float* __restrict__ S, long lds, const 
     for (int i = 0; i < (int)(blockDim.x >> 5); ++i) m = fmaxf(m, red[i]);
     float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < PER; ++i)
-      if (j0 + (int)(threadIdx.x + i * blockDim.x) <= j1) { e[i] = expf(e[i] - m); sum += e[i]; }
-    const float inv = 1.0f / (block_sum_fixed(sum, red) + ((sink || unit_sink) ? expf(sk - m) : 0.f));
-    for (int j = threadIdx.x; j < j0; j += blockDim.x) {
-      P[r * ldp + j] = f2bf(0.f);
-      if (split) P[r * ldp + Sp + j] = f2bf(0.f);
+    for (int i = 0; i < 2 * PER; ++i) {
+      const int j = b0 + 2 * (threadIdx.x + i / 2 * blockDim.x) + (i & 1);
+      e[i] = (j >= j0 && j <= j1) ? expf(e[i] - m) : 0.f;
+      sum += e[i];
     }
+    const float inv = 1.0f / (block_sum_fixed(sum, red) + ((sink || unit_sink) ? expf(sk - m) : 0.f));
+    // the thread's pairs, then the columns on both sides of them
+    auto put = [&](int j, float a, float b) {
+      bf16* d = P + r * ldp + j;
+      const __nv_bfloat162 hi = __floats2bfloat162_rn(a, b);
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(a - __low2float(hi), b - __high2float(hi));
+      if (w2) {
+        *reinterpret_cast<__nv_bfloat162*>(d) = hi;
+        if (split) *reinterpret_cast<__nv_bfloat162*>(d + Sp) = lo;
+      } else {
+        d[0] = __low2bfloat16(hi);
+        if (split) d[Sp] = __low2bfloat16(lo);
+        if (j + 1 < Sp) {
+          d[1] = __high2bfloat16(hi);
+          if (split) d[Sp + 1] = __high2bfloat16(lo);
+        }
+      }
+    };
+    const int end = b0 + 2 * PER * (int)blockDim.x;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      const int j = j0 + threadIdx.x + i * blockDim.x;
-      if (j <= j1) {
-        const float pr = e[i] * inv;
-        const bf16 hi = f2bf(pr);
-        P[r * ldp + j] = hi;
-        if (split) P[r * ldp + Sp + j] = f2bf(pr - bf2f(hi));
-      }
+      const int j = b0 + 2 * (threadIdx.x + i * blockDim.x);
+      if (j < Sp) put(j, e[2 * i] * inv, e[2 * i + 1] * inv);
     }
-    for (int j = j1 + 1 + threadIdx.x; j < Sp; j += blockDim.x) {
-      P[r * ldp + j] = f2bf(0.f);
-      if (split) P[r * ldp + Sp + j] = f2bf(0.f);
-    }
+    for (int j = 2 * threadIdx.x; j < b0; j += 2 * blockDim.x) put(j, 0.f, 0.f);
+    for (int j = end + 2 * threadIdx.x; j < Sp; j += 2 * blockDim.x) put(j, 0.f, 0.f);
     return;
   }
   const float mul = softcap > 0.f ? 1.f : scale;
@@ -1683,19 +1718,26 @@ int b200_lm_linear_state(const float* q, long ldq, const float* k, long ldk, con
   return B200_OK;
 }
 
-int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int dim, void* out, int Kp, int T, void* st) {
-  B200_REQUIRE(q && out && T > 0 && rep > 0 && dim > 0 && Kp >= dim, "lm_heads_to_bf16: bad argument");
-  heads_to_bf16_kernel<<<T * rep, 128, 0, (cudaStream_t)st>>>(q, ldq, rep, dim, (bf16*)out, Kp);
+int b200_lm_heads_to_bf16(const float* q, long ldq, int rep, int G, int dim, void* out, int Kp, int T, void* st) {
+  B200_REQUIRE(q && out && T > 0 && rep > 0 && G > 0 && dim > 0 && Kp >= dim, "lm_heads_to_bf16: bad argument");
+  heads_to_bf16_kernel<<<T * rep, 128, 0, (cudaStream_t)st>>>(q, ldq, rep, G, dim, (bf16*)out, Kp);
+  B200_CHECK_LAUNCH();
+  return B200_OK;
+}
+
+int b200_lm_regroup_heads(const float* x, long ldx, int ldg, int rep, int G, int dv, float* out, long ldo, int T, void* st) {
+  B200_REQUIRE(x && out && T > 0 && rep > 0 && G > 0 && dv > 0 && ldg >= dv, "lm_regroup_heads: bad argument");
+  regroup_heads_kernel<<<T, 256, 0, (cudaStream_t)st>>>(x, ldx, ldg, rep, G, dv, out, ldo);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }
 
 int b200_lm_sink_softmax_bf16(float* S, long lds, const int* pos, int rep, const void* sink, float scale, int chunk,
                               int window, int key0, float bias_exp, int head0, int H, int unit_sink, int split, float softcap, void* P,
-                              long ldp, int rows, int Sp, void* st) {
+                              long ldp, int G, long s_group, long p_group, int rows, int Sp, void* st) {
   B200_REQUIRE(S && pos && P && rows > 0 && rep > 0 && Sp > 0 && key0 >= 0, "lm_sink_softmax_bf16: bad argument");
-  sink_softmax_bf16_kernel<<<rows, 256, 0, (cudaStream_t)st>>>(S, lds, pos, rep, (const bf16*)sink, scale, chunk, window,
-                                                                key0, bias_exp, head0, H > 0 ? H : 1, unit_sink, split, softcap, (bf16*)P, ldp, Sp);
+  sink_softmax_bf16_kernel<<<dim3(rows, G > 1 ? G : 1), 256, 0, (cudaStream_t)st>>>(S, lds, pos, rep, (const bf16*)sink, scale, chunk, window,
+                                                                key0, bias_exp, head0, H > 0 ? H : 1, unit_sink, split, softcap, (bf16*)P, ldp, s_group, p_group, Sp);
   B200_CHECK_LAUNCH();
   return B200_OK;
 }

@@ -667,15 +667,18 @@ int b200_gemm_wt_f32_grouped(const void* X, long ldx, const void* W, long ldw, f
 }
 /* The per-head projections of ONE token set in ONE launch: head g multiplies columns [g * x_group_cols, + n_parts K_w) of
  * X [T, x_cols] (bf16, K_w a multiple of 64; n_parts = 2: [hi | lo] halves of fp32 columns) by W[g] [N, K_w] and writes
- * columns [g * c_group_cols, + N) of C32 [T, ..]. */
+ * columns [g * c_group_cols, + N) of C32 [T, ..].  w_group_cols > 0: W[g] is columns [g * w_group_cols, + K_w) of ONE [N, ..]
+ * matrix (keys of several heads side by side in a cache row); X's groups are then ceil64(K_w) columns, zero beyond K_w. */
 int b200_gemm_wt_f32_heads(const void* X, long ldx, int x_cols, int x_group_cols, const void* W, long ldw, float* C32,
-                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, int n_parts, void* stream) {
-  B200_REQUIRE(X && W && C32 && n_heads > 0 && K_w % 64 == 0 && n_parts >= 1 && x_cols >= (n_heads - 1) * x_group_cols + n_parts * K_w, "gemm_wt_f32_heads: bad argument (K must be whole k-blocks)");
+                           long ldc32, long c_group_cols, int T, int n_heads, int N, int K_w, int n_parts, int w_group_cols, void* stream) {
+  const int kbw = cdiv(K_w, 64);
+  B200_REQUIRE(X && W && C32 && n_heads > 0 && (K_w % 64 == 0 || w_group_cols > 0) && n_parts >= 1 &&
+                   x_cols >= (n_heads - 1) * x_group_cols + n_parts * (w_group_cols > 0 ? kbw * 64 : K_w), "gemm_wt_f32_heads: bad argument (K must be whole k-blocks, or the weights column ranges)");
   WtExt ext;
-  ext.kb_w = K_w / 64; ext.k_w = K_w; ext.ldw = ldw; ext.C32 = C32; ext.res32 = nullptr; ext.ldc32 = ldc32; ext.ldr32 = 0;
-  ext.Csplit = nullptr; ext.ld_split = 0; ext.n_pad = 0;
+  ext.kb_w = kbw; ext.k_w = K_w; ext.ldw = ldw; ext.C32 = C32; ext.res32 = nullptr; ext.ldc32 = ldc32; ext.ldr32 = 0;
+  ext.Csplit = nullptr; ext.ld_split = 0; ext.n_pad = 0; ext.w_group_cols = w_group_cols;
   ext.col_groups = n_heads; ext.x_group_cols = x_group_cols; ext.x_cols = x_cols; ext.c_group_cols = c_group_cols;
-  return gemm_wt_tuned(X, ldx, W, nullptr, nullptr, 0, nullptr, 0, nullptr, 0, T, N, n_parts * K_w, B200_EPI_NONE, B200_WT_F32, 0,
+  return gemm_wt_tuned(X, ldx, W, nullptr, nullptr, 0, nullptr, 0, nullptr, 0, T, N, n_parts * kbw * 64, B200_EPI_NONE, B200_WT_F32, 0,
                        false, 148, nullptr, (cudaStream_t)stream, &ext);
 }
 }

@@ -286,7 +286,7 @@ class LatentAttention:
             for a in range(0, n, step):
                 m = min(step, n - a)
                 qb = ops.to_bf16(qa[a:a + m].view(m * H, Dl), Dl)
-                sc = ops.empty((m * H, S))
+                sc = ops.scores(m * H, S)
                 ops.tc_gemm(qb, rows, sc, N_=S, K=Dl, ldw=rows.stride(0))
                 P = ops.empty((m * H, Sp), torch.bfloat16)
                 ops.masked_softmax_bf16(sc, pos[a:a + m], H, self.scale, P)
@@ -302,7 +302,7 @@ class LatentAttention:
             Sp = (S + 63) // 64 * 64
             ct = ops.cache_transpose(rows[key0:], S, Sp, r)
             qb = ops.to_bf16(qa[a:a + m].view(m * H, Dl), Dl)
-            sc = ops.empty((m * H, S))
+            sc = ops.scores(m * H, S)
             ops.tc_gemm(qb, rows[key0:], sc, N_=S, K=Dl, ldw=rows.stride(0))
             P = ops.empty((m * H, parts * Sp), torch.bfloat16)
             ops.sink_softmax_bf16(sc, pos[a:a + m], H, None, self.scale, 0, self.window, key0, P, split=parts == 2)
@@ -541,7 +541,7 @@ class SinkAttention:
                 for a in range(a0, a0 + m, step):
                     mm = min(step, a0 + m - a)
                     qb16 = ops.heads_to_bf16(q[a:a + mm, g * rep * d:], rep, d)
-                    sc = ops.empty((mm * rep, S))
+                    sc = ops.scores(mm * rep, S)
                     ops.tc_gemm(qb16, keys, sc, N_=S, K=d, ldw=rows.stride(0))
                     P = ops.empty((mm * rep, Sp), torch.bfloat16)
                     ops.sink_softmax_bf16(sc, pos[a:a + mm], rep, self.w["sink"][g * rep:], self.scale, self.chunk, 0, key0, P)
@@ -1231,39 +1231,33 @@ class GroupedAttention:
     def _attend_prompt(self, ctx: StepCtx, q, all_rows, slot_index: int, pos, o, p0: int, n: int):
         """A portion of a prompt (positions p0 .. p0 + n - 1 of one slot) as two tcgen05 products per key/value head:
         the head's cached key columns are the weight-major operand of the scores of the query heads that share it, an
-        fp32 softmax over the visible keys (distance bias and sink included) writes every probability as two bf16 parts
+        fp32 softmax over the visible keys (cap, distance bias and sink included) writes every probability as two bf16 parts
         (the second the rounding error of the first, so the weights keep 16 mantissa bits), and the head's value
-        columns, transposed, are the operand of the weighted sum over both parts.  Queries are taken in chunks that bound the
-        score buffer; with a window a chunk is about a window long and meets only the keys from its first query's
-        first visible key on."""
+        columns, transposed, are the operand of the weighted sum over both parts.  Each step is one launch for all key/value heads.  Queries
+        are taken in chunks, each against the keys from its first query's first visible one to its last query's: half a window
+        of queries (512 without a window), so that most of what is multiplied is seen."""
         ops, H, G, d, dv = ctx.ops, self.H, self.G, self.dim, self.vdim
         rep, rows = H // G, all_rows[slot_index]
-        sink = self.w.get("sink")
-        step = n
-        if self.window:
-            step = max(128, min(self.window, (1 << 27) // (rep * 2 * self.window)))
-            step = -(-n // -(-n // step))          # equal chunks: no short one at the end
+        sink, pitch = self.w.get("sink"), (dv + 3) // 4 * 4
+        step = max(128, self.window // 2 if self.window else 512)
+        longest = min(p0 + n, self.window + step) if self.window else p0 + n
+        step = max(1, min(step, (1 << 27) // (H * longest)))          # bounds the buffer of probabilities
+        step = -(-n // -(-n // step))              # equal chunks: no short one at the end
         for a in range(0, n, step):
             m = min(step, n - a)
             key0 = max(p0 + a - self.window + 1, 0) if self.window else 0
             S = p0 + a + m - key0
             Sp = (S + 63) // 64 * 64
-            sub = max(1, min(m, (1 << 27) // (rep * Sp)))
-            for g in range(G):
-                keys = rows[key0:key0 + S, g * d:(g + 1) * d]
-                vt = ops.cache_transpose(rows[key0:, G * d + g * dv:], S, Sp, dv)
-                for b in range(a, a + m, sub):
-                    mm = min(sub, a + m - b)
-                    qb16 = ops.heads_to_bf16(q[b:b + mm, g * rep * d:], rep, d)
-                    sc = ops.empty((mm * rep, S))
-                    ops.tc_gemm(qb16, keys, sc, N_=S, K=d, ldw=rows.stride(0))
-                    P = ops.empty((mm * rep, 2 * Sp), torch.bfloat16)
-                    ops.sink_softmax_bf16(sc, pos[b:b + mm], rep, None if sink is None else sink[g * rep:], self.scale, 0,
-                                          self.window, key0, P, bias_exp=self.bias_exp, head0=g * rep, H=H,
-                                          unit_sink=self.sink == "unit", split=True, softcap=self.softcap)
-                    og = ops.empty((mm * rep, dv))
-                    ops.tc_gemm(P, vt, og, N_=dv, K=Sp, parts=2)
-                    ops.head_post(og.view(mm, rep * dv), o[b:b + mm, g * rep * dv:(g + 1) * rep * dv], dv=dv)
+            vt = ops.cache_transpose(rows[key0:, G * d:], S, Sp, G * dv)
+            qb16 = ops.heads_to_bf16(q[a:a + m], rep, d, G)
+            sc, P = ops.empty((m * rep, G * Sp)), ops.empty((m * rep, G * 2 * Sp), torch.bfloat16)
+            ops.tc_gemm_heads(qb16, rows[key0:], sc, H=G, N_=S, K=d, x_cols=qb16.shape[1], x_group_cols=qb16.shape[1] // G,
+                              c_group_cols=Sp, w_group_cols=d, ldw=rows.stride(0))
+            ops.sink_softmax_bf16(sc, pos[a:a + m], rep, sink, self.scale, 0, self.window, key0, P, bias_exp=self.bias_exp, head0=0, H=H,
+                                  unit_sink=self.sink == "unit", split=True, softcap=self.softcap, G=G)
+            og = ops.empty((m * rep, G * pitch))
+            ops.tc_gemm_heads(P, vt, og, H=G, N_=dv, K=Sp, x_cols=G * 2 * Sp, x_group_cols=2 * Sp, c_group_cols=pitch, parts=2)
+            ops.regroup_heads(og, rep, G, dv, o[a:a + m])
 
 
 class TokenShiftState:

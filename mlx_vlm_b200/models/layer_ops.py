@@ -421,11 +421,13 @@ class LayerOps:
                                                    N_, K, self.s), "gemm_wt_f32_grouped")
 
     def tc_gemm_heads(self, Xb: torch.Tensor, W: torch.Tensor, Y: torch.Tensor, *, H: int, N_: int, K: int,
-                      x_cols: int, x_group_cols: int, c_group_cols: int, parts: int = 1):
+                      x_cols: int, x_group_cols: int, c_group_cols: int, parts: int = 1, w_group_cols: int = 0, ldw: Optional[int] = None):
         """Y[:, g * c_group_cols : + N_] = Xb[:, g * x_group_cols : + K] . W[g]^T for every head g, ONE tcgen05 launch;
-        parts = 2: a head's columns are the [hi | lo] halves of K fp32 numbers"""
-        self._ok(self.lib.b200_gemm_wt_f32_heads(Xb.data_ptr(), Xb.stride(0), x_cols, x_group_cols, W.data_ptr(), K,
-                                                 Y.data_ptr(), Y.stride(0), c_group_cols, Xb.shape[0], H, N_, K, int(parts), self.s),
+        parts = 2: a head's columns are the [hi | lo] halves of K fp32 numbers; w_group_cols: W[g] is columns g * w_group_cols : + K
+        of one matrix (row pitch ldw)"""
+        self._ok(self.lib.b200_gemm_wt_f32_heads(Xb.data_ptr(), Xb.stride(0), x_cols, x_group_cols, W.data_ptr(),
+                                                 K if ldw is None else ldw, Y.data_ptr(), Y.stride(0), c_group_cols, Xb.shape[0], H, N_, K,
+                                                 int(parts), int(w_group_cols), self.s),
                  "gemm_wt_f32_heads")
 
     def rows_scatter(self, X: torch.Tensor, dst_map: torch.Tensor, out: torch.Tensor, rows: int):
@@ -579,22 +581,33 @@ class LayerOps:
             float(softcap), N.ptr(part), n_split, T, self.s),
             "lm_sink_attention")
 
-    def heads_to_bf16(self, q: torch.Tensor, rep: int, dim: int) -> torch.Tensor:
-        """q (n, >= rep * dim) fp32 columns of `rep` heads -> bf16 rows (n * rep, ceil64(dim))"""
+    def heads_to_bf16(self, q: torch.Tensor, rep: int, dim: int, G: int = 1) -> torch.Tensor:
+        """q (n, >= G * rep * dim) fp32 columns of G groups of `rep` heads -> bf16 rows (n * rep, G * ceil64(dim))"""
         n, Kp = q.shape[0], (dim + 63) // 64 * 64
-        out = self.empty((n * rep, Kp), torch.bfloat16)
-        self._ok(self.lib.b200_lm_heads_to_bf16(q.data_ptr(), q.stride(0), rep, dim, out.data_ptr(), Kp, n, self.s),
+        out = self.empty((n * rep, G * Kp), torch.bfloat16)
+        self._ok(self.lib.b200_lm_heads_to_bf16(q.data_ptr(), q.stride(0), rep, int(G), dim, out.data_ptr(), Kp, n, self.s),
                  "lm_heads_to_bf16")
         return out
 
+    def regroup_heads(self, x: torch.Tensor, rep: int, G: int, dv: int, out: torch.Tensor):
+        """x (T rep, G pitch): rows (t, r), the dv numbers of head g rep + r in the columns of group g -> out (T, G rep dv)"""
+        self._ok(self.lib.b200_lm_regroup_heads(x.data_ptr(), x.stride(0), x.shape[1] // G, rep, G, dv, out.data_ptr(), out.stride(0),
+                                                out.shape[0], self.s), "lm_regroup_heads")
+
+    def scores(self, rows: int, S: int) -> torch.Tensor:
+        """(rows, S) fp32 scratch whose rows start on 16-byte boundaries"""
+        return self.empty((rows, (S + 63) // 64 * 64))[:, :S]
+
     def sink_softmax_bf16(self, S, pos, rep, sink, scale, chunk, window, key0, P, bias_exp: float = 0.0, head0: int = 0,
-                          H: int = 1, unit_sink: bool = False, split: bool = False, softcap: float = 0.0):
+                          H: int = 1, unit_sink: bool = False, split: bool = False, softcap: float = 0.0, G: int = 1):
         """head0, H: the first head of the rows' group and the number of heads (they fix the slopes of the distance bias);
-        split: P (rows, 2 Sp) gets every probability as two bf16 parts [hi | lo], the operand of `tc_gemm(parts=2)`"""
+        split: P (rows, 2 Sp) gets every probability as two bf16 parts [hi | lo], the operand of `tc_gemm(parts=2)`;
+        G: S and P hold the rows of G groups of `rep` heads side by side in equal parts of their columns"""
         self._ok(self.lib.b200_lm_sink_softmax_bf16(S.data_ptr(), S.stride(0), pos.data_ptr(), rep, N.ptr(sink), float(scale),
                                                     int(chunk), int(window), int(key0), float(bias_exp), int(head0), int(H),
-                                                    int(unit_sink), int(split), float(softcap), P.data_ptr(), P.stride(0),
-                                                    S.shape[0], P.shape[1] // 2 if split else P.shape[1], self.s),
+                                                    int(unit_sink), int(split), float(softcap), P.data_ptr(), P.stride(0), int(G),
+                                                    S.shape[1] // G, P.shape[1] // G, S.shape[0],
+                                                    P.shape[1] // G // 2 if split else P.shape[1] // G, self.s),
                  "lm_sink_softmax_bf16")
 
     def linear_state(self, q, k, v, out, state, ctx, *, H, rep, dim, vdim, act=False, unit_eps=0.0, q_scale=1.0,
