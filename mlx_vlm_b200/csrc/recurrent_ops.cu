@@ -382,7 +382,7 @@ __device__ __forceinline__ void tile_product_staged(MemTile& tile, const float (
 }
 
 template <bool VEC>
-__global__ void __launch_bounds__(MC_THREADS) memory_chunk_kernel(MemP p) {
+__global__ void __launch_bounds__(MC_THREADS, 4) memory_chunk_kernel(MemP p) {
   __shared__ MemTile tile;
   __shared__ float ws[MC];
   const int seq = blockIdx.z, h = blockIdx.y, d = p.dim, dv = p.vdim;
